@@ -370,6 +370,83 @@ int ytcuda_qwen3_tp_resync(void* handle);
  * says. len > max_position_embeddings returns YTC_UNSUPPORTED. */
 int ytcuda_qwen3_forward(void* handle, const int32_t* ids, int len, float* logits, void* stream);
 
+/* ---------------------------------------------------------------- language-model mechanisms outside the reference
+ * Operators of the models below that YTensor has no counterpart for, each usable on its own. */
+
+/* Causal attention over a sliding window with capped scores and a K/V ring. q_len queries per sequence at positions
+ * pos0 .. pos0 + q_len - 1; position p lies in ring row p % ring of k / v [batch, kv_heads, ring, dim], where the new
+ * positions have already been stored. A query sees the last `window` positions up to itself (0: all);
+ * score = scale * q.k, then softcap * tanh(score / softcap) when softcap > 0. Strides {batch, head, row} in elements.
+ * bf16 with head_dim == value_dim in {64, 128} and a ring of whole 128-row tiles runs on tcgen05. */
+int ytcuda_window_attn_fwd(int dtype, const void* q, const void* k, const void* v, void* o, int batch, int kv_heads,
+                           int groups, int q_len, int head_dim, int value_dim, const int64_t* q_strides,
+                           const int64_t* k_strides, const int64_t* v_strides, const int64_t* o_strides, int64_t pos0,
+                           int window, int ring, float scale, float softcap, void* stream);
+
+/* Router of a mixture of experts with `identity` identity experts behind the `experts` real ones: s = softmax(logits)
+ * over all of them, choice scores s + correction; of `groups` equal groups of neighbours only the `keep` whose largest
+ * choice score is best can be chosen; the `top` largest choice scores are, with weights s (not renormalised).
+ * choice / weight [rows, top] in the order of choice (-1: none left); rank [rows, top]: running number of the token
+ * among its expert's tokens; count [experts] is increased by the arrivals (the caller zeroes it). */
+int ytcuda_moe_route(const float* logits, int64_t row_stride, const float* correction, int64_t rows, int experts,
+                     int identity, int top, int groups, int keep, int32_t* choice, float* weight, int32_t* rank,
+                     int32_t* count, void* stream);
+
+/* Residual stream around a sublayer: x += y / rms(y) * w_post (skipped when w_post is NULL), then
+ * h = x / rms(x) * w_pre in fp32 or bf16 (skipped when w_pre is NULL); rms(v) = sqrt(mean(v^2) + eps) over the first
+ * `width` of row_stride channels. One launch. */
+int ytcuda_residual_norm(float* x, const float* y, const float* w_post, const float* w_pre, void* h, int dtype, int64_t rows,
+                         int width, int row_stride, float eps, void* stream);
+
+/* y[m, n] = act(x[m, k] . W[n, k]^T), W bf16, x and y bf16 (tensor cores) or fp32 (FFMA). act 0: none, 1: exact (erf)
+ * gelu, 2: the rows of W alternate gate_j, up_j and y[m, n / 2] = silu(gate) * up. With block_group, rows come in blocks
+ * of 128 and block i uses matrix block_group[i] of `groups` stacked ones (-1: the block is passed over). */
+int ytcuda_linear_act(int dtype, int act, const void* x, int64_t x_row_stride, const void* w_bf16, void* y,
+                      int64_t y_row_stride, int m, int n, int k, const int32_t* block_group, int groups, void* stream);
+
+/* ---------------------------------------------------------------- Duzozen decoder
+ * Decoder-only model: norm before and after each sublayer, sliding-window attention with capped scores, values mixed
+ * with the first mixing layer's, dense (erf gelu) or mixture-of-experts (silu-gated) feed-forward. Sizes are padded by
+ * the caller (zero weights): width, head dims and feed-forward widths are multiples of 8, norms run over norm_width. */
+#define YTC_MLP_NONE 0
+#define YTC_MLP_DENSE 1
+#define YTC_MLP_MOE 2
+typedef struct {
+  int width, norm_width, vocab, layers;
+  int batch;      /* sequences, all of one length */
+  int max_tokens; /* longest sequence */
+  int chunk;      /* most tokens per sequence that run through the layers at once */
+  int dtype;      /* YTC_BF16: bf16 activations and cache, fp32 residual stream; YTC_F32: everything fp32 */
+  float eps;
+} ytcuda_duzozen_config;
+typedef struct {
+  int heads, kv_heads, dim, vdim;
+  int window; /* 0: unlimited */
+  int v_mix;
+  int mlp; /* YTC_MLP_* */
+  int ff;
+  int experts, identity, top, groups, keep; /* YTC_MLP_MOE; groups = keep = 1: no groups */
+  float scale;
+  float softcap; /* 0: none */
+} ytcuda_duzozen_layer;
+/* Returns NULL on an unsupported configuration (see ytcuda_last_error_string). */
+void* ytcuda_duzozen_create(const ytcuda_duzozen_config* cfg, const ytcuda_duzozen_layer* layers);
+void ytcuda_duzozen_destroy(void* handle);
+/* Registers a device weight (borrowed). "embed", "head" [vocab, width] bf16, "norm" [width] fp32; per layer fp32
+ * "norm1", "norm1b", "norm2", "norm2b" [width], "vmix" [1], "correction" [experts + identity]; bf16 "qkv" [q heads, k
+ * heads, v heads; width], "o" [width, heads * vdim], "up" / "down" [ff, width] / [width, ff] (dense) or [experts, 2 ff,
+ * width] with gate_j, up_j alternating / [experts, width, ff], "router" [experts + identity, width]. */
+int ytcuda_duzozen_set_weight(void* handle, const char* name, int layer, const void* dptr);
+int ytcuda_duzozen_reset(void* handle);
+int64_t ytcuda_duzozen_cache_len(void* handle);
+/* One new token of a single sequence: 0 = the graph of fused decode kernels, 1 = one launch per operator as for longer
+ * inputs. */
+int ytcuda_duzozen_set_decode_path(void* handle, int path);
+/* Appends ids [batch, len] (device) to the sequences. want (HOST, n_want distinct row numbers in [0, batch * len), in
+ * the order of the tokens) selects the rows whose logits [n_want, vocab] (device, fp32) are computed. */
+int ytcuda_duzozen_forward(void* handle, const int32_t* ids, int len, const int32_t* want, int n_want, float* logits,
+                           void* stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -73,6 +73,18 @@ SIGNATURES = {
     "ytcuda_qwen3_tp_disconnect": (_i, [_vp]),
     "ytcuda_qwen3_tp_resync": (_i, [_vp]),
     "ytcuda_qwen3_forward": (_i, [_vp, _vp, _i, _vp, _vp]),
+    "ytcuda_window_attn_fwd": (_i, [_i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i64, _i, _i, _f,
+                                    _f, _vp]),
+    "ytcuda_moe_route": (_i, [_vp, _i64, _vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp]),
+    "ytcuda_residual_norm": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i64, _i, _i, _f, _vp]),
+    "ytcuda_linear_act": (_i, [_i, _i, _vp, _i64, _vp, _vp, _i64, _i, _i, _i, _vp, _i, _vp]),
+    "ytcuda_duzozen_create": (_vp, [_vp, _vp]),
+    "ytcuda_duzozen_destroy": (None, [_vp]),
+    "ytcuda_duzozen_set_weight": (_i, [_vp, C.c_char_p, _i, _vp]),
+    "ytcuda_duzozen_reset": (_i, [_vp]),
+    "ytcuda_duzozen_cache_len": (_i64, [_vp]),
+    "ytcuda_duzozen_set_decode_path": (_i, [_vp, _i]),
+    "ytcuda_duzozen_forward": (_i, [_vp, _vp, _i, _vp, _i, _vp, _vp]),
 }
 
 
@@ -87,6 +99,9 @@ class YtCudaInvalidArgument(YtCudaError, ValueError):
 
 
 _lib = None
+# False in a process that asked for the library of one model only (registry.load_model(build=True)): entry points that
+# library does not hold are then missing from lib() and fail when they are called.
+full_library = True
 
 
 def lib() -> C.CDLL:
@@ -98,7 +113,12 @@ def lib() -> C.CDLL:
                 "(there is no CPU fallback)")
         L = C.CDLL(str(LIB_PATH))
         for name, (res, args) in SIGNATURES.items():
-            fn = getattr(L, name)
+            try:
+                fn = getattr(L, name)
+            except AttributeError:  # a library built for one model holds no other model's entry points
+                if full_library:
+                    raise
+                continue
             fn.restype = res
             fn.argtypes = args
         _lib = L

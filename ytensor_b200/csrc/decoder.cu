@@ -10,7 +10,7 @@
 // numbers). Tensor parallelism splits heads and FFN columns over ranks; the partial sums after the attention
 // output projection and after the down projection are reduced by a callback the caller provides (NCCL all-reduce).
 //
-// Kernels here: embedding gather; weight-streaming linear for few rows (decode); fp32 -> (hi, lo) bf16 split that
+// Kernels here (the embedding gather is in lm_rows.cu): weight-streaming linear for few rows (decode); fp32 -> (hi, lo) bf16 split that
 // lets the tcgen05 GEMM multiply fp32 activations by bf16 weights (prefill); fused per-head RMSNorm + RoPE + KV
 // append; argmax partials for a vocabulary split over ranks.
 #include <math_constants.h>
@@ -28,28 +28,6 @@
 #include "ytc_common.cuh"
 
 namespace ytk {
-
-// ------------------------------------------------------------------ embedding gather
-// out[t, :] = float(table[ids[t], :])   (reference qwen3.cpp:378-385)
-__global__ void __launch_bounds__(256) embedding_kernel(const uint16_t* table, const int* ids, float* out, int64_t n,
-                                                        int hidden, int vocab) {
-  const int per_row = hidden / 4;
-  const int64_t total = n * per_row;
-  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
-       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-    const int64_t t = i / per_row;
-    const int c = static_cast<int>(i - t * per_row) * 4;
-    int id = ids[t];
-    id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
-    const uint2 w = *reinterpret_cast<const uint2*>(table + static_cast<int64_t>(id) * hidden + c);
-    float4 o;
-    o.x = bf16_bits_to_f32(static_cast<uint16_t>(w.x & 0xFFFF));
-    o.y = bf16_bits_to_f32(static_cast<uint16_t>(w.x >> 16));
-    o.z = bf16_bits_to_f32(static_cast<uint16_t>(w.y & 0xFFFF));
-    o.w = bf16_bits_to_f32(static_cast<uint16_t>(w.y >> 16));
-    *reinterpret_cast<float4*>(out + t * hidden + c) = o;
-  }
-}
 
 // ------------------------------------------------------------------ few-row linear (decode)
 // y[m, n] (+)= sum_k x[m, k] * float(W[n, k]),  m < M <= MT. One warp owns ROWS weight rows and streams them once
@@ -685,21 +663,6 @@ int ytcuda_rope_tables(int dim, int max_len, float theta, float* cos_host, float
       cos_host[static_cast<int64_t>(t) * dim + i] = cos_host[static_cast<int64_t>(t) * dim + i + half] = std::cos(angle);
       sin_host[static_cast<int64_t>(t) * dim + i] = sin_host[static_cast<int64_t>(t) * dim + i + half] = std::sin(angle);
     }
-  return YTC_OK;
-}
-
-int ytcuda_embedding(const void* table_bf16, const int32_t* ids, float* out, int64_t n, int hidden, int vocab,
-                     void* stream) {
-  YTC_REQUIRE(n >= 0 && hidden >= 0 && vocab > 0, "ytcuda_embedding: bad extent");
-  if (n == 0 || hidden == 0) return YTC_OK;
-  YTC_REQUIRE(table_bf16 && ids && out, "ytcuda_embedding: null tensor");
-  YTC_REQUIRE(hidden % 4 == 0, "ytcuda_embedding: hidden must be a multiple of 4");
-  const int64_t blocks = (n * (hidden / 4) + 255) / 256;
-  const int64_t cap = static_cast<int64_t>(sm_count()) * 16;
-  embedding_kernel<<<static_cast<unsigned>(blocks < cap ? blocks : cap), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const uint16_t*>(table_bf16), ids, out, n, hidden, vocab);
-  count_launch();
-  YTC_CUDA(cudaGetLastError());
   return YTC_OK;
 }
 

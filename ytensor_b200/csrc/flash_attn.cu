@@ -12,6 +12,9 @@
 //  * attn_simt_kernel : any dtype (fp32 included), any head / value dim, one warp per query row. The
 //                       catch-all for shapes the tensor-core kernel does not take.
 //
+// Sliding windows, capped scores and K/V rings (window_attention, the windowed language models) are forms of the same
+// kernels: flash_tc_kernel<D, FA_WINDOW / FA_WINDOW_BOUNDED> and attn_simt_kernel.
+//
 // Both honour: no mask / causal window anchored at the end of the keys / a bool mask [q_len, kv_len];
 // an optional additive fp32 bias [q_len, kv_len]; rows that see no key produce zeros.
 // Replaces yt::function::scaledDotProductAttention and yt::kernel::avx2::flash_attention
@@ -21,6 +24,7 @@
 #include <atomic>
 #include <type_traits>
 
+#include "lm_ops.cuh"
 #include "ptx_sm100.cuh"
 #include "ytc_common.cuh"
 
@@ -52,7 +56,18 @@ struct FlashParams {
   int n_items;               // row_blocks * items_per_row_block
   uint32_t idesc_s, idesc_pv;
   int* status;
+  // windowed forms: key index 0 is position 128 * key_tile0, tile j of the keys lies in ring rows
+  // ((key_tile0 + j) % ring_tiles) * 128 .., row r sees key c iff r + causal_off - window < c <= r + causal_off
+  int window, key_tile0, ring_tiles;
+  float cap_log2;            // softcap * log2(e), 0 = scores are not capped
+  float cap_in;              // 2 * log2(e) * scale / softcap: 2^(raw * cap_in) = exp(2 * scale * raw / softcap)
 };
+
+// FA_PLAIN: the general kernel. FA_WINDOW: sliding window over a K/V ring, scores optionally capped.
+// FA_WINDOW_BOUNDED: as FA_WINDOW with scores capped so low (|score| <= FA_BOUNDED_CAP) that exp(score - cap) cannot
+// underflow: the cap itself is the softmax reference, so there is no running maximum and O is never rescaled.
+enum { FA_PLAIN = 0, FA_WINDOW = 1, FA_WINDOW_BOUNDED = 2 };
+constexpr float FA_BOUNDED_CAP = 40.f;
 
 // 2^x by the special-function unit (ex2.approx.ftz): -inf gives 0, relative error about 2^-22.
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -118,6 +133,13 @@ __device__ __forceinline__ void exp2_emu2(uint64_t x2, float& p0, float& p1) {
   p1 = __int_as_float(__float_as_int(q1) + (__float_as_int(t1) << 23));
 }
 
+// 1 / x by the special-function unit (rcp.approx.ftz, relative error about 2^-23; 1 / inf = 0).
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <int D>
 struct FaSmem {
   static constexpr int TILE_BYTES = FA_BM * D * 2;  // one Q / K / V tile
@@ -146,9 +168,11 @@ __device__ __forceinline__ void fa_load_tile(uint8_t* dst, const CUtensorMap* m,
 struct FaItem {
   int q_head[2], q_row0[2], kv_head, b;
   bool tile_on[2];
-  int n_tiles[2], n_max;
+  int n_tiles[2], n_max;  // end (exclusive) of the key tiles of each query tile, and of both
+  int j0;                 // first key tile of both (0 without a window)
 };
 
+template <int MODE>
 __device__ __forceinline__ FaItem fa_decode_item(const FlashParams& p, int w) {
   FaItem it;
   const int per_rb = p.items_per_row_block;
@@ -181,10 +205,15 @@ __device__ __forceinline__ FaItem fa_decode_item(const FlashParams& p, int w) {
     it.n_tiles[t] = (!it.tile_on[t] || last_key < 0) ? 0 : last_key / FA_BN + 1;
   }
   it.n_max = it.n_tiles[0] > it.n_tiles[1] ? it.n_tiles[0] : it.n_tiles[1];
+  it.j0 = 0;
+  if (MODE != FA_PLAIN) {  // (query tile 0 holds the lower rows, whose window reaches furthest back)
+    const int first = it.q_row0[0] + p.causal_off - p.window + 1;
+    it.j0 = first > 0 ? first / FA_BN : 0;
+  }
   return it;
 }
 
-template <int D>
+template <int D, int MODE>
 __global__ void __launch_bounds__(FA_THREADS, 1)
     flash_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const FlashParams p) {
@@ -241,6 +270,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
   // tensor-memory columns: S0/P0 at 0, S1/P1 at 128, O0 at 256, O1 at 384
   const uint32_t t_s[2] = {tmem_base, tmem_base + 128u};
   const uint32_t t_o[2] = {tmem_base + 256u, tmem_base + 384u};
+  dependent_wait();  // (set-up done in shared and tensor memory; global memory may be touched from here on)
+  dependent_trigger();
 
   if (warp == 0) {
     // ------------------------------------------------------------ TMA producer
@@ -249,8 +280,8 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
       bool ok = true;
       int n_item = 0;
       for (int w = blockIdx.x; ok && w < p.n_items; w += gridDim.x) {
-        const FaItem it = fa_decode_item(p, w);
-        if (it.n_max == 0) continue;  // nothing visible: the softmax warpgroups write zeros on their own
+        const FaItem it = fa_decode_item<MODE>(p, w);
+        if (it.n_max <= it.j0) continue;  // nothing visible: the softmax warpgroups write zeros on their own
         // (n_item counts only items with work; items without work touch no barrier in any role)
         if (n_item > 0 && !mbar_wait(q_free, static_cast<uint32_t>((n_item - 1) & 1), abort_word)) break;
         int n_q = 0;
@@ -259,7 +290,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
         for (int t = 0; t < 2; ++t)
           if (it.tile_on[t])
             fa_load_tile<D>(smem + S::Q_OFF + t * S::TILE_BYTES, &tmQ, q_full, it.q_row0[t], it.q_head[t], it.b);
-        for (int j = 0; j < it.n_max; ++j, ++kv_cnt) {
+        for (int j = it.j0; j < it.n_max; ++j, ++kv_cnt) {
           const int s = kv_cnt % FA_STAGES;
           if (!mbar_wait(&kv_empty[s], static_cast<uint32_t>(((kv_cnt / FA_STAGES) & 1) ^ 1), abort_word)) {
             ok = false;
@@ -268,9 +299,10 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
           uint8_t* ks = smem + S::KV_OFF + s * 2 * S::TILE_BYTES;
           uint8_t* vs = ks + S::TILE_BYTES;
           mbar_expect_tx(&k_full[s], S::TILE_BYTES);
-          fa_load_tile<D>(ks, &tmK, &k_full[s], j * FA_BN, it.kv_head, it.b);
+          const int key_row = (MODE == FA_PLAIN ? j : (p.key_tile0 + j) % p.ring_tiles) * FA_BN;
+          fa_load_tile<D>(ks, &tmK, &k_full[s], key_row, it.kv_head, it.b);
           mbar_expect_tx(&v_full[s], S::TILE_BYTES);
-          fa_load_tile<D>(vs, &tmV, &v_full[s], j * FA_BN, it.kv_head, it.b);
+          fa_load_tile<D>(vs, &tmV, &v_full[s], key_row, it.kv_head, it.b);
         }
         ++n_item;
       }
@@ -316,15 +348,15 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
       bool ok = true;
       int n_item = 0;
       for (int w = blockIdx.x; ok && w < p.n_items; w += gridDim.x) {
-        const FaItem it = fa_decode_item(p, w);
-        if (it.n_max == 0) continue;
+        const FaItem it = fa_decode_item<MODE>(p, w);
+        if (it.n_max <= it.j0) continue;
         if (!mbar_wait(q_full, static_cast<uint32_t>(n_item & 1), abort_word)) break;
         if (!mbar_wait(&k_full[kv_cnt % FA_STAGES], static_cast<uint32_t>((kv_cnt / FA_STAGES) & 1), abort_word)) break;
         tc_fence_after();
-        if (it.n_tiles[0] > 0) issue_s(0, kv_cnt % FA_STAGES);
-        if (it.n_tiles[1] > 0) issue_s(1, kv_cnt % FA_STAGES);
-        if (it.n_max == 1) tc_commit(q_free);
-        for (int j = 0; j < it.n_max && ok; ++j, ++kv_cnt) {
+        if (it.n_tiles[0] > it.j0) issue_s(0, kv_cnt % FA_STAGES);
+        if (it.n_tiles[1] > it.j0) issue_s(1, kv_cnt % FA_STAGES);
+        if (it.n_max == it.j0 + 1) tc_commit(q_free);
+        for (int j = it.j0; j < it.n_max && ok; ++j, ++kv_cnt) {
           const int s = kv_cnt % FA_STAGES;
           const int sn = (kv_cnt + 1) % FA_STAGES;
           const uint32_t ph = static_cast<uint32_t>((kv_cnt / FA_STAGES) & 1);
@@ -340,20 +372,20 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
                 ok = false;
                 break;
               }
-              if (j == 0 && e_cnt[t] > 0 &&
+              if (j == it.j0 && e_cnt[t] > 0 &&
                   !mbar_wait(&o_free[t], static_cast<uint32_t>((e_cnt[t] - 1) & 1), abort_word)) {
                 ok = false;  // the first P.V of an item overwrites O_t: the previous epilogue must have read it
                 break;
               }
               tc_fence_after();
-              issue_pv(t, s, j > 0, 0);
+              issue_pv(t, s, j > it.j0, 0);
               if (!mbar_wait(&p_full[t], static_cast<uint32_t>(p_cnt[t] & 1), abort_word)) {
                 ok = false;
                 break;
               }
               ++p_cnt[t];
               tc_fence_after();
-              issue_pv(t, s, j > 0, 1);
+              issue_pv(t, s, j > it.j0, 1);
             }
             if (j + 1 < it.n_tiles[t]) {
               if (!mbar_wait(&k_full[sn], ph_next, abort_word)) {
@@ -369,7 +401,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
           tc_commit(&kv_empty[s]);  // every MMA that read stage s has been issued before this point
         }
         for (int t = 0; t < 2; ++t)
-          if (it.n_tiles[t] > 0) ++e_cnt[t];
+          if (it.n_tiles[t] > it.j0) ++e_cnt[t];
         ++n_item;
       }
     }
@@ -384,13 +416,14 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
     int s_base = 0;  // S tiles (= P tiles = P.V products) of this query tile in earlier items
     bool ok = true;
     for (int w = blockIdx.x; ok && w < p.n_items; w += gridDim.x) {
-      const FaItem it = fa_decode_item(p, w);
+      const FaItem it = fa_decode_item<MODE>(p, w);
       const int* q_row0 = it.q_row0;
       const int* q_head = it.q_head;
       const bool* tile_on = it.tile_on;
       const int b = it.b;
       const int row = q_row0[t] + row_in_tile;  // global query row
-      const int nt = (it.n_max == 0) ? 0 : it.n_tiles[t];
+      const int j0 = MODE == FA_PLAIN ? 0 : it.j0;
+      const int nt = (it.n_tiles[t] <= j0) ? 0 : it.n_tiles[t] - j0;  // key tiles of this query tile
       const int o_base = s_base;
       float m_run = -CUDART_INF_F;  // running maximum, log2 domain
       float l_run = 0.f;
@@ -401,14 +434,116 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
           break;
         }
         tc_fence_after();
-        const int key0 = j * FA_BN;
+        const int key0 = (j0 + j) * FA_BN;
         // Three kinds of tile: `full` (every key visible to every row), limited (visibility is "key <= per-row
         // limit": causal diagonal, end of the keys, rows past q_len), general (bool mask or bias present).
         int row_limit = (row < p.q_len) ? p.kv_len - 1 : -1;
         if (p.causal && row + p.causal_off < row_limit) row_limit = row + p.causal_off;
         const int cl = row_limit - key0;  // columns 0..cl of this tile are visible to this thread's row
         const bool full = !elementwise_mask && (key0 + FA_BN <= p.kv_len) && (q_row0[t] + FA_BM <= p.q_len) &&
-                          (!p.causal || key0 + FA_BN - 1 <= q_row0[t] + p.causal_off);
+                          (!p.causal || key0 + FA_BN - 1 <= q_row0[t] + p.causal_off) &&
+                          (MODE == FA_PLAIN || key0 >= q_row0[t] + FA_BM + p.causal_off - p.window);
+        if constexpr (MODE != FA_PLAIN) {
+          // Columns cw .. cl of the tile are visible to this thread's row.
+          const int cw = row + p.causal_off - p.window + 1 - key0;
+          const bool capped = MODE == FA_WINDOW_BOUNDED || p.cap_log2 > 0.f;
+          // the score in log2 units is cap * tanh(x) = cap - 2 cap / (1 + exp(2 x)) with x = scale * raw / softcap
+          const float two_cap = -2.f * p.cap_log2;
+          float shift = 0.f;  // what is added to the log2 score: minus the softmax reference (here: the cap itself)
+          if constexpr (MODE == FA_WINDOW) {
+            float mx = -CUDART_INF_F;  // (the cap is monotonic: the maximum is taken over the raw scores)
+            const bool pos = p.scale_log2 >= 0.f;
+#pragma unroll 1
+            for (int c0 = 0; c0 < FA_BN; c0 += 32) {
+              if (!full && __all_sync(0xffffffffu, cl < c0 || cw > c0 + 31)) continue;
+              uint32_t r[32];
+              tmem_ld_32x32b_x32(ts + c0, r);
+              tmem_ld_wait();
+#pragma unroll
+              for (int e = 0; e < 32; ++e) {
+                const float v = pos ? __uint_as_float(r[e]) : -__uint_as_float(r[e]);
+                mx = (full || (c0 + e <= cl && c0 + e >= cw)) ? fmaxf(mx, v) : mx;
+              }
+            }
+            if (mx != -CUDART_INF_F) {
+              const float raw = pos ? mx : -mx;
+              mx = capped ? p.cap_log2 + two_cap * fast_rcp(1.f + fast_exp2(raw * p.cap_in)) : raw * p.scale_log2;
+            }
+            const float m_new = fmaxf(m_run, mx);
+            if (j == 0) {
+              m_run = m_new;
+            } else if (__any_sync(0xffffffffu, (m_new - m_run) > FA_RESCALE_THRESHOLD)) {
+              // O_t *= 2^(m_run - m_new) for this warp's 32 rows; needs the previous P.V to have landed
+              if (!mbar_wait(&o_ready[t], static_cast<uint32_t>((o_base + j - 1) & 1), abort_word)) {
+                ok = false;
+                break;
+              }
+              tc_fence_after();
+              const float alpha = (m_new == -CUDART_INF_F) ? 1.f : fast_exp2(m_run - m_new);
+#pragma unroll 1
+              for (int c0 = 0; c0 < D; c0 += 16) {
+                uint32_t r[16];
+                tmem_ld_32x32b_x16(to + c0, r);
+                tmem_ld_wait();
+#pragma unroll
+                for (int e = 0; e < 16; ++e) r[e] = __float_as_uint(__uint_as_float(r[e]) * alpha);
+                tmem_st_32x32b_x16(to + c0, r);
+              }
+              l_run *= alpha;
+              m_run = m_new;
+            }
+            shift = (m_run == -CUDART_INF_F) ? 0.f : -m_run;
+            if (capped) shift += p.cap_log2;
+          }
+          float l0 = 0.f, l1 = 0.f;
+#pragma unroll 1
+          for (int c0 = 0; c0 < FA_BN; c0 += 64) {
+            uint32_t pk[32];
+            const bool dead = !full && __all_sync(0xffffffffu, cl < c0 || cw > c0 + 63);
+            if (dead) {
+#pragma unroll
+              for (int e = 0; e < 32; ++e) pk[e] = 0u;
+            } else {
+              uint32_t r[64];
+              tmem_ld_32x32b_x64(ts + c0, r);
+              tmem_ld_wait();
+              const int hi = full ? 64 : cl - c0, lo = full ? 0 : cw - c0;
+              auto body = [&](auto is_capped) {
+#pragma unroll
+                for (int e = 0; e < 64; e += 2) {
+                  float v[2];
+#pragma unroll
+                  for (int u = 0; u < 2; ++u) {
+                    const float raw = __uint_as_float(r[e + u]);
+                    float x;
+                    if (decltype(is_capped)::value) x = fmaf(two_cap, fast_rcp(1.f + fast_exp2(raw * p.cap_in)), shift);
+                    else x = fmaf(raw, p.scale_log2, shift);
+                    v[u] = fast_exp2(x);
+                    v[u] = (e + u <= hi && e + u >= lo) ? v[u] : 0.f;
+                  }
+                  l0 += v[0];
+                  l1 += v[1];
+                  pk[e >> 1] = pack_bf16x2_rn(v[0], v[1]);
+                }
+              };
+              if (capped) body(std::true_type{});
+              else body(std::false_type{});
+            }
+            tmem_st_32x32b_x32(ts + (c0 >> 1), pk);
+            if (c0 == 0) {  // the columns of P for keys 0..63 are stored: the MMA warp may start P.V on them
+              tmem_st_wait();
+              tc_fence_before();
+              __syncwarp();
+              if (lane == 0) mbar_arrive(&p_half[t]);
+            }
+          }
+          l_run += l0 + l1;
+          tmem_st_wait();
+          tc_fence_before();
+          __syncwarp();
+          if (lane == 0) mbar_arrive(&p_full[t]);
+          continue;
+        }
         auto score = [&](uint32_t raw, int c) -> float {  // general tiles only
           float v = __uint_as_float(raw) * p.scale_log2;
           const int key = key0 + c;
@@ -638,6 +773,10 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
 #pragma unroll
             for (int e = 0; e < 32; e += 2) {
               const float a0 = __uint_as_float(r[e]) * inv, a1 = __uint_as_float(r[e + 1]) * inv;
+              if (MODE != FA_PLAIN) {
+                w[e >> 1] = pack_bf16x2_rn(a0, a1);
+                continue;
+              }
               const uint16_t lo = p.is_bf16 ? f32_to_bf16_bits_ref(a0) : f32_to_f16_bits_ref(a0);
               const uint16_t hi = p.is_bf16 ? f32_to_bf16_bits_ref(a1) : f32_to_f16_bits_ref(a1);
               w[e >> 1] = static_cast<uint32_t>(lo) | (static_cast<uint32_t>(hi) << 16);
@@ -689,12 +828,17 @@ struct AttnSimtParams {
   int causal, causal_off;
   float scale;
   int dt;
+  int window = 0;     // > 0: row r sees only the last `window` keys up to r + causal_off
+  int ring = 0;       // > 0: key c lies in row c % ring of K and V
+  float softcap = 0;  // > 0: score <- softcap * tanh(score / softcap)
 };
 
 constexpr int SIMT_MAX_D = 256;
 
 __global__ void __launch_bounds__(128) attn_simt_kernel(const AttnSimtParams p) {
   __shared__ float q_s[4][SIMT_MAX_D];
+  dependent_wait();
+  dependent_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int heads = p.kv_heads * p.groups;
   const int64_t total_rows = static_cast<int64_t>(p.batch) * heads * p.q_len;
@@ -716,16 +860,19 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const AttnSimtParams p) 
     float m_run = -CUDART_INF_F, l_run = 0.f;
     int last = p.kv_len - 1;
     if (p.causal && row + p.causal_off < last) last = row + p.causal_off;
-    for (int k0 = 0; k0 <= last; k0 += 32) {
+    int first = 0;
+    if (p.window > 0 && row + p.causal_off - p.window + 1 > 0) first = row + p.causal_off - p.window + 1;
+    for (int k0 = first; k0 <= last; k0 += 32) {
       const int key = k0 + lane;
       bool vis = key <= last;
       if (vis && p.mask) vis = p.mask[static_cast<int64_t>(row) * p.mask_rs + key] != 0;
       float s = -CUDART_INF_F;
       if (vis) {
         float dot = 0.f;
-        const int64_t kb = ko + static_cast<int64_t>(key) * p.k_sr;
+        const int64_t kb = ko + static_cast<int64_t>(p.ring > 0 ? key % p.ring : key) * p.k_sr;
         for (int i = 0; i < p.d; ++i) dot = fmaf(q_s[warp][i], load_as_f32(p.K, kb + i, p.dt), dot);
         s = dot * p.scale;
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
         if (p.bias) s += p.bias[static_cast<int64_t>(row) * p.bias_rs + key * p.bias_cs];
       }
       float mx = s;
@@ -746,7 +893,7 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const AttnSimtParams p) 
       for (int kk = 0; kk < nk; ++kk) {
         const float pk = __shfl_sync(0xffffffffu, pr, kk);
         if (pk == 0.f) continue;
-        const int64_t vb = vo + static_cast<int64_t>(k0 + kk) * p.v_sr;
+        const int64_t vb = vo + static_cast<int64_t>(p.ring > 0 ? (k0 + kk) % p.ring : k0 + kk) * p.v_sr;
 #pragma unroll
         for (int i = 0; i < SIMT_MAX_D / 32; ++i) {
           const int c = i * 32 + lane;
@@ -759,7 +906,9 @@ __global__ void __launch_bounds__(128) attn_simt_kernel(const AttnSimtParams p) 
 #pragma unroll
     for (int i = 0; i < SIMT_MAX_D / 32; ++i) {
       const int c = i * 32 + lane;
-      if (c < p.dv) store_from_f32(p.O, oo + c, acc[i] * inv, p.dt);
+      if (c >= p.dv) continue;
+      if (p.ring > 0 && p.dt == YTC_BF16) static_cast<uint16_t*>(p.O)[oo + c] = bf16_rn_bits(acc[i] * inv);
+      else store_from_f32(p.O, oo + c, acc[i] * inv, p.dt);
     }
   }
 }
@@ -1460,6 +1609,102 @@ static bool tc_strides_ok(const void* ptr, int64_t s_row, int64_t s_head, int64_
   return true;
 }
 
+template <int D>
+static int launch_window_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FlashParams& p,
+                            bool bounded, cudaStream_t st) {
+  const dim3 grid(static_cast<unsigned>(p.n_items < sm_count() ? p.n_items : sm_count()));
+  auto* fn = bounded ? flash_tc_kernel<D, FA_WINDOW_BOUNDED> : flash_tc_kernel<D, FA_WINDOW>;
+  const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(fn), FaSmem<D>::DYN_BYTES);
+  if (s != YTC_OK) return s;
+  YTC_CUDA(launch_overlapped(fn, grid, dim3(FA_THREADS), FaSmem<D>::DYN_BYTES, st, tmQ, tmK, tmV, p));
+  count_launch();
+  YTC_CUDA(cudaGetLastError());
+  return YTC_OK;
+}
+
+int window_attention(const WindowAttn& a, cudaStream_t st) {
+  const int heads = a.kv_heads * a.groups;
+  const int64_t end = a.pos0 + a.q_len;  // keys 0 .. end - 1 have been appended
+  const int64_t oldest = (a.window > 0 && a.pos0 - a.window + 1 > 0) ? a.pos0 - a.window + 1 : 0;
+  YTC_REQUIRE(a.batch > 0 && a.kv_heads > 0 && a.groups > 0 && a.q_len > 0 && a.ring > 0 && a.window >= 0,
+              "window_attention: bad extent");
+  YTC_REQUIRE(end - oldest <= a.ring && end <= 0x7fffffff, "window_attention: a ring of %d rows does not hold the keys of "
+              "positions %lld .. %lld", a.ring, static_cast<long long>(oldest), static_cast<long long>(end - 1));
+  const bool tc = a.dtype == YTC_BF16 && a.head_dim == a.value_dim && (a.head_dim == 64 || a.head_dim == 128) &&
+                  a.ring % FA_BN == 0 && end - oldest / FA_BN * FA_BN <= a.ring && g_attn_path != 1 &&
+                  tc_strides_ok(a.q, a.q_st[2], a.q_st[1], a.q_st[0], a.q_len, heads, a.batch) &&
+                  tc_strides_ok(a.k, a.k_st[2], a.k_st[1], a.k_st[0], a.ring, a.kv_heads, a.batch) &&
+                  tc_strides_ok(a.v, a.v_st[2], a.v_st[1], a.v_st[0], a.ring, a.kv_heads, a.batch) &&
+                  (reinterpret_cast<uint64_t>(a.o) & 3u) == 0 && a.o_st[0] % 2 == 0 && a.o_st[1] % 2 == 0 &&
+                  a.o_st[2] % 2 == 0;
+  if (tc) {
+    CUtensorMap tmQ, tmK, tmV;
+    int s = make_qkv_map(&tmQ, a.q, a.head_dim, a.q_len, heads, a.batch, a.q_st[2], a.q_st[1], a.q_st[0]);
+    if (s != YTC_OK) return s;
+    if ((s = make_qkv_map(&tmK, a.k, a.head_dim, a.ring, a.kv_heads, a.batch, a.k_st[2], a.k_st[1], a.k_st[0])) != YTC_OK)
+      return s;
+    if ((s = make_qkv_map(&tmV, a.v, a.value_dim, a.ring, a.kv_heads, a.batch, a.v_st[2], a.v_st[1], a.v_st[0])) != YTC_OK)
+      return s;
+    FlashParams p{};
+    p.O = a.o;
+    p.o_sb = a.o_st[0]; p.o_sh = a.o_st[1]; p.o_sr = a.o_st[2];
+    p.batch = a.batch; p.kv_heads = a.kv_heads; p.groups = a.groups; p.q_len = a.q_len;
+    p.key_tile0 = static_cast<int>(oldest / FA_BN);
+    p.ring_tiles = a.ring / FA_BN;
+    const int base = p.key_tile0 * FA_BN;  // key index 0 of this call
+    p.kv_len = static_cast<int>(end) - base;
+    p.causal = 1;
+    p.causal_off = static_cast<int>(a.pos0) - base;
+    p.window = a.window > 0 ? a.window : 0x3fffffff;
+    p.scale_log2 = a.scale * FA_LOG2E;
+    p.cap_log2 = a.softcap > 0.f ? a.softcap * FA_LOG2E : 0.f;
+    p.cap_in = a.softcap > 0.f ? 2.f * FA_LOG2E * a.scale / a.softcap : 0.f;
+    p.is_bf16 = 1;
+    p.pair_heads = (a.groups % 2 == 0) ? 1 : 0;
+    p.idesc_s = umma_idesc(1u, 0, 0, FA_BM, FA_BN);
+    p.idesc_pv = umma_idesc(1u, 0, 1, FA_BM, static_cast<uint32_t>(a.value_dim));
+    p.status = device_status_word();
+    if (!p.status) {
+      set_last_error("window_attention: no device status word");
+      return YTC_CUDA_ERROR;
+    }
+    p.row_blocks = p.pair_heads ? (a.q_len + FA_BM - 1) / FA_BM : (a.q_len + 2 * FA_BM - 1) / (2 * FA_BM);
+    p.head_slots = p.pair_heads ? heads / 2 : heads;
+    const int64_t items = static_cast<int64_t>(p.row_blocks) * p.head_slots * a.batch;
+    if (items > 0x7fffffffll) {
+      set_last_error("window_attention: too many work items");
+      return YTC_UNSUPPORTED;
+    }
+    p.items_per_row_block = p.head_slots * a.batch;
+    p.n_items = static_cast<int>(items);
+    const bool bounded = a.softcap > 0.f && a.softcap <= FA_BOUNDED_CAP;
+    return a.head_dim == 128 ? launch_window_tc<128>(tmQ, tmK, tmV, p, bounded, st)
+                             : launch_window_tc<64>(tmQ, tmK, tmV, p, bounded, st);
+  }
+  if (a.head_dim > SIMT_MAX_D || a.value_dim > SIMT_MAX_D) {
+    set_last_error("window_attention: head_dim / value_dim above %d are not supported", SIMT_MAX_D);
+    return YTC_UNSUPPORTED;
+  }
+  AttnSimtParams p{};
+  p.Q = a.q; p.K = a.k; p.V = a.v; p.O = a.o;
+  p.q_sb = a.q_st[0]; p.q_sh = a.q_st[1]; p.q_sr = a.q_st[2];
+  p.k_sb = a.k_st[0]; p.k_sh = a.k_st[1]; p.k_sr = a.k_st[2];
+  p.v_sb = a.v_st[0]; p.v_sh = a.v_st[1]; p.v_sr = a.v_st[2];
+  p.o_sb = a.o_st[0]; p.o_sh = a.o_st[1]; p.o_sr = a.o_st[2];
+  p.batch = a.batch; p.kv_heads = a.kv_heads; p.groups = a.groups; p.q_len = a.q_len;
+  p.kv_len = static_cast<int>(end);
+  p.d = a.head_dim; p.dv = a.value_dim;
+  p.causal = 1; p.causal_off = static_cast<int>(a.pos0);
+  p.scale = a.scale; p.dt = a.dtype;
+  p.window = a.window; p.ring = a.ring; p.softcap = a.softcap;
+  const int64_t rows = static_cast<int64_t>(a.batch) * heads * a.q_len;
+  const int64_t blocks = (rows + 3) / 4, cap = static_cast<int64_t>(sm_count()) * 16;
+  YTC_CUDA(launch_overlapped(attn_simt_kernel, dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)), dim3(128), 0, st, p));
+  count_launch();
+  YTC_CUDA(cudaGetLastError());
+  return YTC_OK;
+}
+
 }  // namespace ytk
 
 using namespace ytk;
@@ -1519,6 +1764,8 @@ int ytcuda_flash_attn_fwd(int dtype, const void* Q, const void* K, const void* V
     p.batch = batch; p.kv_heads = kv_heads; p.groups = groups; p.q_len = q_len; p.kv_len = kv_len;
     p.causal = causal; p.causal_off = causal_offset;
     p.scale_log2 = scale * FA_LOG2E;
+    p.window = p.key_tile0 = p.ring_tiles = 0;
+    p.cap_log2 = p.cap_in = 0.f;
     p.is_bf16 = dtype == YTC_BF16;
     p.pair_heads = (groups % 2 == 0) ? 1 : 0;
     const uint32_t fmt = dtype == YTC_BF16 ? 1u : 0u;
@@ -1545,13 +1792,13 @@ int ytcuda_flash_attn_fwd(int dtype, const void* Q, const void* K, const void* V
     p.n_items = static_cast<int>(items);
     const dim3 grid(static_cast<unsigned>(p.n_items < sm_count() ? p.n_items : sm_count()));
     if (head_dim == 128) {
-      const int sa = ensure_dynamic_smem(reinterpret_cast<const void*>(flash_tc_kernel<128>), FaSmem<128>::DYN_BYTES);
+      const int sa = ensure_dynamic_smem(reinterpret_cast<const void*>(flash_tc_kernel<128, FA_PLAIN>), FaSmem<128>::DYN_BYTES);
       if (sa != YTC_OK) return sa;
-      flash_tc_kernel<128><<<grid, FA_THREADS, FaSmem<128>::DYN_BYTES, st>>>(tmQ, tmK, tmV, p);
+      flash_tc_kernel<128, FA_PLAIN><<<grid, FA_THREADS, FaSmem<128>::DYN_BYTES, st>>>(tmQ, tmK, tmV, p);
     } else {
-      const int sa = ensure_dynamic_smem(reinterpret_cast<const void*>(flash_tc_kernel<64>), FaSmem<64>::DYN_BYTES);
+      const int sa = ensure_dynamic_smem(reinterpret_cast<const void*>(flash_tc_kernel<64, FA_PLAIN>), FaSmem<64>::DYN_BYTES);
       if (sa != YTC_OK) return sa;
-      flash_tc_kernel<64><<<grid, FA_THREADS, FaSmem<64>::DYN_BYTES, st>>>(tmQ, tmK, tmV, p);
+      flash_tc_kernel<64, FA_PLAIN><<<grid, FA_THREADS, FaSmem<64>::DYN_BYTES, st>>>(tmQ, tmK, tmV, p);
     }
     count_launch();
     YTC_CUDA(cudaGetLastError());

@@ -12,6 +12,7 @@
 // src/kernel/avx2/hgemm.inl:139-288) behind ytcuda_gemm.
 #include <atomic>
 
+#include "lm_ops.cuh"
 #include "ptx_sm100.cuh"
 #include "ytc_common.cuh"
 
@@ -40,6 +41,12 @@ struct GemmTcParams {
   // masked product: tile_live[mb * tiles_n + nb] == 0 marks an output tile no element of which is asked for; every
   // role of the kernel passes over it (no loads, no MMAs, no stores). NULL = every tile is computed.
   const uint8_t* tile_live;
+  // linear layers of the language models (LinearEpilogue, lm_ops.cuh)
+  int epi;                 // EPI_NONE: the store rules above; otherwise tc_store_epilogue
+  // grouped product: every 128-row block of A belongs to one group (expert) or to none (-1, passed over); group g
+  // multiplies rows g * group_rows .. of the stacked B operand. NULL = ordinary product.
+  const int* tile_group;
+  int group_rows;
 };
 
 template <int BN>
@@ -125,6 +132,52 @@ __device__ __forceinline__ void tc_store_chunk(const GemmTcParams& p, const uint
         DType<OUT_DT>::store(p.C, idx, v);
       }
     }
+  }
+}
+
+// Store with a fused activation and round-to-nearest-even narrowing (see LinearEpilogue). One thread holds 32
+// consecutive columns of one row; EPI_SWIGLU_PAIRS makes 16 results of them.
+__device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const uint32_t (&r)[32], int64_t row_off, int gn0,
+                                                  bool row_ok) {
+  if (!row_ok) return;
+  if (p.epi == EPI_SWIGLU_PAIRS) {
+    uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + (gn0 >> 1);
+    uint32_t w[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      const float a = lm_silu_fast(__uint_as_float(r[4 * j])) * __uint_as_float(r[4 * j + 1]);
+      const float b = lm_silu_fast(__uint_as_float(r[4 * j + 2])) * __uint_as_float(r[4 * j + 3]);
+      w[j] = pack_bf16x2_rn(a, b);
+    }
+    if (gn0 + 32 <= p.N && (reinterpret_cast<uint64_t>(dst) & 15u) == 0) {
+      reinterpret_cast<uint4*>(dst)[0] = make_uint4(w[0], w[1], w[2], w[3]);
+      reinterpret_cast<uint4*>(dst)[1] = make_uint4(w[4], w[5], w[6], w[7]);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 16; ++j)
+        if (gn0 + 2 * j + 1 < p.N) dst[j] = static_cast<uint16_t>(w[j >> 1] >> ((j & 1) * 16));
+    }
+    return;
+  }
+  uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + gn0;
+  uint32_t w[16];
+#pragma unroll
+  for (int j = 0; j < 16; ++j) {
+    float a = __uint_as_float(r[2 * j]), b = __uint_as_float(r[2 * j + 1]);
+    if (p.epi == EPI_GELU_ERF) {
+      a = lm_gelu_erf(a);
+      b = lm_gelu_erf(b);
+    }
+    w[j] = pack_bf16x2_rn(a, b);
+  }
+  if (gn0 + 32 <= p.N && (reinterpret_cast<uint64_t>(dst) & 15u) == 0) {
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      reinterpret_cast<uint4*>(dst)[j] = make_uint4(w[4 * j], w[4 * j + 1], w[4 * j + 2], w[4 * j + 3]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      if (gn0 + j < p.N) dst[j] = static_cast<uint16_t>(w[j >> 1] >> ((j & 1) * 16));
   }
 }
 
@@ -216,6 +269,9 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
         if (p.tile_live && !p.tile_live[rem]) continue;
         const int mb = rem / p.tiles_n;
         const int nb = rem - mb * p.tiles_n;
+        const int group = p.tile_group ? p.tile_group[mb] : 0;
+        if (group < 0) continue;
+        const int n_row0 = group * p.group_rows + nb * BN;
         const int ba = p.a_bcast ? 0 : b;
         const int bb = p.b_bcast ? 0 : b;
         for (int kb = 0; kb < p.k_blocks; ++kb) {
@@ -250,14 +306,14 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
             if (p.split_loads) {
 #pragma unroll
               for (int c = 0; c < BN / 64; ++c)
-                tma_load_3d(sb + c * 8192, &tmB, &full_bar[stage], kb * TC_BK, nb * BN + c * 64, bb);
+                tma_load_3d(sb + c * 8192, &tmB, &full_bar[stage], kb * TC_BK, n_row0 + c * 64, bb);
             } else {
-              tma_load_3d(sb, &tmB, &full_bar[stage], kb * TC_BK, nb * BN, bb);
+              tma_load_3d(sb, &tmB, &full_bar[stage], kb * TC_BK, n_row0, bb);
             }
           } else {
 #pragma unroll
             for (int c = 0; c < BN / 64; ++c)
-              tma_load_3d(sb + c * 8192, &tmB, &full_bar[stage], nb * BN + c * 64, kb * TC_BK, bb);
+              tma_load_3d(sb + c * 8192, &tmB, &full_bar[stage], n_row0 + c * 64, kb * TC_BK, bb);
           }
           ++issued;
           if (++stage == TC_STAGES) {
@@ -292,6 +348,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
       bool ok = true;
       for (int tile = blockIdx.x; ok && tile < p.total_tiles; tile += gridDim.x) {
         if (p.tile_live && !p.tile_live[tile % tiles_per_batch]) continue;
+        if (p.tile_group && p.tile_group[(tile % tiles_per_batch) / p.tiles_n] < 0) continue;
         if (!mbar_wait(&tempty_bar[acc], acc_phase ^ 1u, abort_word)) break;
         tc_fence_after();
         const uint32_t d_tmem = tmem_base + static_cast<uint32_t>(acc * BN);
@@ -337,6 +394,7 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
       if (p.tile_live && !p.tile_live[rem]) continue;
       const int mb = rem / p.tiles_n;
       const int nb = rem - mb * p.tiles_n;
+      if (p.tile_group && p.tile_group[mb] < 0) continue;
       if (!mbar_wait(&tfull_bar[acc], acc_phase, abort_word)) break;
       tc_fence_after();
       const int gm = mb * TC_BM + row;
@@ -353,7 +411,8 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
         tmem_ld_wait();
         const int gn0 = nb * BN + c0;
         if (gn0 < p.N) {
-          if (p.out_dtype == YTC_BF16) tc_store_chunk<BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
+          if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
+          else if (p.out_dtype == YTC_BF16) tc_store_chunk<BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
           else if (p.out_dtype == YTC_F32) tc_store_chunk<BN, YTC_F32>(p, r, row_off, gn0, row_ok, vec_ok);
           else tc_store_chunk<BN, YTC_F16>(p, r, row_off, gn0, row_ok, vec_ok);
         }
@@ -558,7 +617,8 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
         tmem_ld_wait();
         const int gn0 = nb * TC2_BN + c0;
         if (gn0 < p.N) {
-          if (p.out_dtype == YTC_BF16) tc_store_chunk<TC2_BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
+          if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
+          else if (p.out_dtype == YTC_BF16) tc_store_chunk<TC2_BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
           else if (p.out_dtype == YTC_F32) tc_store_chunk<TC2_BN, YTC_F32>(p, r, row_off, gn0, row_ok, vec_ok);
           else tc_store_chunk<TC2_BN, YTC_F16>(p, r, row_off, gn0, row_ok, vec_ok);
         }
@@ -792,7 +852,8 @@ static int make_tile_live(int m, int n, int bm, int bn, cudaStream_t st, uint8_t
 
 static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, void* C, int m, int n, int k,
                      float alpha, float beta, int a_mn, int64_t lda, int b_mn, int64_t ldb, int64_t rsc, int64_t csc,
-                     int64_t batch, int64_t bsa, int64_t bsb, int64_t bsc, cudaStream_t st) {
+                     int64_t batch, int64_t bsa, int64_t bsb, int64_t bsc, cudaStream_t st,
+                     const LinearEpilogue* ex = nullptr) {
   // A: unit axis = K (a_mn 0, dims {K, M}) or M (a_mn 1, dims {M, K}). B likewise with N.
   CUtensorMap tmA, tmB;
   const int a_bcast = (batch > 1 && bsa == 0) ? 1 : 0;
@@ -801,7 +862,8 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
   const int BN = (n <= 128 || static_cast<int64_t>((m + 127) / 128) * ((n + 255) / 256) * batch < sm_count() / 2) ? 128 : 256;
   // CTA pairs pay off on large problems; small ones keep one CTA per tile (more tiles to spread over the SMs)
   // (a masked product keeps one CTA per tile: the tile-skipping form of the kernel)
-  const bool pair = g_mask.kind == 0 && g_tc_pair != 2 &&
+  const bool grouped = ex && ex->tile_group;
+  const bool pair = g_mask.kind == 0 && g_tc_pair != 2 && !grouped &&
                     (g_tc_pair == 1 || (m >= 512 && n >= 256 && k >= 256 &&
                                         static_cast<int64_t>((m + 255) / 256) * ((n + 255) / 256) * batch >= 74));
   {
@@ -822,7 +884,8 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
     const uint64_t nb = (b_bcast || batch == 1) ? 1 : static_cast<uint64_t>(batch);
     uint64_t dims[3], strides[2];
     uint32_t box[3];
-    if (!b_mn) { dims[0] = k; dims[1] = n; box[0] = TC_BK; box[1] = pair ? 128u : (g_tc_split_loads ? 64u : static_cast<uint32_t>(BN)); }
+    const uint64_t b_rows = grouped ? static_cast<uint64_t>(n) * ex->groups : static_cast<uint64_t>(n);
+    if (!b_mn) { dims[0] = k; dims[1] = b_rows; box[0] = TC_BK; box[1] = pair ? 128u : (g_tc_split_loads ? 64u : static_cast<uint32_t>(BN)); }
     else       { dims[0] = n; dims[1] = k; box[0] = 64;    box[1] = TC_BK; }
     dims[2] = nb;
     box[2] = 1;
@@ -852,6 +915,10 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
   p.k_blocks = (k + TC_BK - 1) / TC_BK;
   p.a_prefetch = g_tc_a_prefetch;
   p.split_loads = g_tc_split_loads;
+  p.tile_live = nullptr;
+  p.epi = ex ? ex->epi : EPI_NONE;
+  p.tile_group = grouped ? ex->tile_group : nullptr;
+  p.group_rows = n;
   p.status = device_status_word();
   if (!p.status) {
     set_last_error("ytcuda_gemm: no device status word");
@@ -893,6 +960,19 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
   if (live) cudaFreeAsync(live, st);
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
+}
+
+// y[m, n] = epilogue(x[m, k] . W[n, k]^T) on the tensor cores (lm_ops.cuh).
+int linear_tc(const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, int64_t ldy, int out_dtype, int m, int n,
+              int k, const LinearEpilogue& ex, cudaStream_t st) {
+  if (m <= 0 || n <= 0) return YTC_OK;
+  int unused;
+  YTC_REQUIRE(tc_operand_ok(x, ldx, 1, 0, 1, m, k, &unused) && tc_operand_ok(w, ldw, 1, 0, 1, n, k, &unused),
+              "linear_tc: operand rows must be 16-byte aligned");
+  YTC_REQUIRE(ex.epi == EPI_NONE || out_dtype == YTC_BF16, "linear_tc: fused epilogues store bf16");
+  YTC_REQUIRE(ex.epi != EPI_SWIGLU_PAIRS || n % 2 == 0, "linear_tc: an odd number of gate / up rows");
+  YTC_REQUIRE(!ex.tile_group || m % TC_BM == 0, "linear_tc: grouped rows come in blocks of %d", TC_BM);
+  return launch_tc(YTC_BF16, out_dtype, x, w, y, m, n, k, 1.f, 0.f, 0, ldx, 0, ldw, ldy, 1, 1, 0, 0, 0, st, &ex);
 }
 
 static int launch_simt(int dtype_in, int dtype_out, const void* A, const void* B, void* C, int m, int n, int k,

@@ -14,6 +14,7 @@ import numpy as np
 
 from . import _lib
 from ._lib import check, lib
+from .causal_lm import CausalLM
 
 
 @dataclass
@@ -103,7 +104,7 @@ def shard_weight(cfg: Qwen3Config, name: str, w: np.ndarray, rank: int, world: i
 _ALLREDUCE_T = C.CFUNCTYPE(C.c_int, C.c_void_p, C.c_int64, C.c_void_p)
 
 
-class Qwen3ForCausalLM:
+class Qwen3ForCausalLM(CausalLM):
     """Device model for `batch` sequences; rank `tp_rank` of `tp_world` tensor-parallel ranks."""
 
     def __init__(self, cfg: Qwen3Config, batch: int = 1, tp_rank: int = 0, tp_world: int = 1, group=None,
@@ -226,12 +227,12 @@ class Qwen3ForCausalLM:
     def argmax(self, logits):
         """Greedy token per sequence (global over the tensor-parallel group): value / index pairs of the local
         maxima are all-gathered and the first global maximum wins, as a host argmax over the full row would."""
+        if self.tp_world == 1:
+            return super().argmax(logits)
         from . import api
         torch = self.torch
         val, idx = api.max(logits, -1)
         idx = idx.reshape(-1) + self.v0
-        if self.tp_world == 1:
-            return idx.to(torch.int32), val.reshape(-1)
         import torch.distributed as dist
         vals = [torch.empty_like(val.reshape(-1)) for _ in range(self.tp_world)]
         idxs = [torch.empty_like(idx) for _ in range(self.tp_world)]
@@ -242,13 +243,9 @@ class Qwen3ForCausalLM:
         tok = torch.stack(idxs, 1).gather(1, which.reshape(-1, 1).long()).reshape(-1)
         return tok.to(torch.int32), best.reshape(-1)
 
-    def check_status(self) -> None:
-        """Reads the device status word (synchronises the stream). A bounded wait that ran out - under tensor
-        parallelism: a peer that never arrived at an exchange - raises; the KV caches are then half written and the
-        group has to call recover() before the next forward."""
-        st = self.L.ytcuda_device_status(self.torch.cuda.current_stream().cuda_stream)
-        if st != _lib.OK:
-            raise _lib.YtCudaError(st, _lib.last_error() or "a bounded device-side wait ran out")
+    @property
+    def can_sample(self) -> bool:  # sampling needs the whole vocabulary on one GPU
+        return self.tp_world == 1
 
     def recover(self) -> None:
         """After check_status raised on some rank: EVERY rank of the group calls this. Kernels are waited for,
@@ -261,39 +258,6 @@ class Qwen3ForCausalLM:
             dist.barrier(group=self.group)
         else:
             self.reset_kv_cache()
-
-    def generate_greedy(self, prompt_ids, steps: int):
-        """prompt_ids int32 [batch, len] (device). Returns int32 [batch, steps] greedy tokens. The device status is
-        checked once at the end, so that a step kernel that gave up on a peer raises instead of yielding tokens."""
-        torch = self.torch
-        out = torch.empty(self.batch, steps, dtype=torch.int32, device=prompt_ids.device)
-        logits = self.forward(prompt_ids)
-        for s in range(steps):
-            tok, _ = self.argmax(logits)
-            out[:, s] = tok
-            if s + 1 < steps:
-                logits = self.forward(tok.reshape(self.batch, 1).contiguous())
-        self.check_status()
-        return out
-
-    def generate_topk(self, prompt_ids, steps: int, k: int = 20, seed: int = 42):
-        """Sampled generation as Qwen3ForCausalLM::generate does it (reference qwen3.cpp:459-516): after every
-        forward the next token is drawn among the k most probable ones. The uniform numbers come from a host
-        generator (numpy's MT19937 seeded with `seed`; the reference's std::uniform_real_distribution consumes its
-        std::mt19937 differently, so the streams are not the same). Single GPU. Returns int32 [batch, steps]."""
-        from . import api
-        torch = self.torch
-        assert self.tp_world == 1, "sampling needs the whole vocabulary on one GPU"
-        rng = np.random.Generator(np.random.MT19937(seed))
-        out = torch.empty(self.batch, steps, dtype=torch.int32, device=prompt_ids.device)
-        logits = self.forward(prompt_ids)
-        for s in range(steps):
-            u = torch.from_numpy(rng.random(self.batch, dtype=np.float32)).to(prompt_ids.device)
-            _, _, tok = api.topk_sample(logits, k, u)
-            out[:, s] = tok
-            if s + 1 < steps:
-                logits = self.forward(tok.reshape(self.batch, 1).contiguous())
-        return out
 
     def close(self):
         """Destroys the model. Under tensor parallelism every rank must call it (it runs a barrier over the group
