@@ -27,6 +27,7 @@ Prints ONE JSON line on rank 0.
 from __future__ import annotations
 
 import argparse
+import ctypes
 import json
 import os
 import statistics
@@ -201,7 +202,9 @@ def _cpu_backend():
         be = O.ref(threads=cores)
         cores = be.threads()
     else:
-        be, cores = O.port(), 1
+        be = O.port()
+        # (a launcher that starts several ranks sets OMP_NUM_THREADS to 1; the CPU arm runs on rank 0 alone)
+        ctypes.CDLL("libgomp.so.1").omp_set_num_threads(cores)
     return be, kind, cores
 
 
@@ -329,7 +332,8 @@ def reference_arm(args) -> None:
     if int(os.environ.get("RANK", "0")) != 0:
         return
     world = int(os.environ.get("WORLD_SIZE", "1"))
-    items = 4
+    from oracle import oracle as O
+    items = 4 if O.ref_available() else 1  # (the plain-C restatement is an order of magnitude slower)
     runs = []
     for _ in range(max(1, min(args.steps, 3))):
         runs.append(cpu_gemm(budget_s=0.0, items=items))
