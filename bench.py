@@ -17,6 +17,8 @@ roofline, end-to-end (host buffers) and CPU-baseline legs:
   chain     rmsNorm + broadcast residual + row softmax + bf16 cast on [32,4096,4096] fp32   (N = 1 only)
   gemm32    fp32 GEMM 1024^3                                                                (N = 1 only)
   gemm_weak the headline GEMM with 64 matrices PER RANK                                     (N > 1 only)
+`--workload lm` (on request only): prefill and decode throughput of the Duzozen model at a few sizes, beside the Qwen3
+decoder of equal size.
 Every secondary workload runs in a child process of its own (same rank environment, its own rendezvous port), so a
 failure there is recorded in its entry and cannot take the headline with it.
 
@@ -35,6 +37,7 @@ import subprocess
 import sys
 import threading
 import time
+import zlib
 from pathlib import Path
 
 ROOT = Path(__file__).resolve().parent
@@ -817,8 +820,164 @@ def decode_arm(args) -> list | None:
     return results if D.rank == 0 else None
 
 
+# ======================================================================================= windowed model
+def _device_weights(torch, shapes, seed=4, std=0.02):
+    """name -> random bf16 tensor on the device, made when it is asked for."""
+    class W:
+        def __getitem__(self, name):
+            g = torch.Generator(device="cuda").manual_seed(seed + zlib.crc32(name.encode()))
+            shape = shapes[name]
+            if "norm" in name:
+                return torch.ones(shape, dtype=torch.bfloat16, device="cuda")
+            if name.endswith("vmix"):
+                return torch.full(shape, 0.5, dtype=torch.bfloat16, device="cuda")
+            return (torch.randn(shape, generator=g, device="cuda") * std).to(torch.bfloat16)
+    return W()
+
+
+def lm_sizes():
+    """Layers of the size of a real model: name -> (Duzozen configuration, Qwen3 configuration of equal size)."""
+    from ytensor_b200 import qwen3 as Q
+    from ytensor_b200.duzozen import MLP_DENSE, MLP_MOE, DuzozenConfig, DuzozenLayer
+
+    def make(width, vocab, n, heads, kv, window, **mlp):
+        att = dict(heads=heads, kv_heads=kv, dim=128, vdim=128, scale=128 ** -0.5, softcap=20.0, window=window, v_mix=True)
+        dense = dict(mlp=MLP_DENSE, ff=mlp["dense"])
+        rest = dict(mlp=MLP_MOE, **mlp["moe"]) if "moe" in mlp else dense
+        return DuzozenConfig(width=width, vocab=vocab, eps=1e-6,
+                             layers=[DuzozenLayer(**att, **(rest if l else dense)) for l in range(n)])
+
+    small = Q.Qwen3Config(max_position_embeddings=8192)
+    large = Q.Qwen3Config(hidden_size=4096, num_hidden_layers=8, vocab_size=32768, intermediate_size=9600,
+                          num_attention_heads=32, num_key_value_heads=8, max_position_embeddings=8192)
+    return {
+        "width 1024, 28 layers, dense": (make(1024, 151936, 28, 16, 8, 1024, dense=4608), small),
+        "width 1024, 28 layers, 64 experts + 8 identity, top 8": (
+            make(1024, 151936, 28, 16, 8, 1024, dense=4608,
+                 moe=dict(ff=384, experts=64, identity=8, top=8, groups=8, keep=4)), small),
+        "width 4096, 8 layers, dense": (make(4096, 32768, 8, 32, 8, 2048, dense=14400), large),
+        "width 4096, 8 layers, 32 experts + 4 identity, top 4": (
+            make(4096, 32768, 8, 32, 8, 2048, dense=14400,
+                 moe=dict(ff=2400, experts=32, identity=4, top=4, groups=6, keep=3)), large),
+    }
+
+
+def lm_arm(args) -> list | None:
+    """Prefill and decode throughput of the Duzozen model at a few sizes beside the Qwen3 decoder of equal size (random
+    weights; one GPU, one sequence). Prefill: prompts of 512 and 4096 tokens; decode: 128 single-token steps behind the
+    4096-token prompt (the Qwen3 decoder: also behind 512). Device time by CUDA events."""
+    D = Dist()
+    torch = D.torch
+    from ytensor_b200 import qwen3 as Q
+    from ytensor_b200.duzozen import MLP_DENSE, MLP_MOE, DuzozenForCausalLM
+    peaks = measured_peaks()
+    reps = max(3, min(args.steps, 5))
+
+    def measure(m, vocab, lens, steps=128):
+        ids = torch.randint(0, vocab, (1, max(lens)), dtype=torch.int32, device=D.dev)
+        out = {}
+        for n in lens:
+            ts, ds = [], []
+            for rep in range(reps + 2):
+                m.reset_kv_cache()
+                ev = [torch.cuda.Event(enable_timing=True) for _ in range(3)]
+                prompt = ids[:, :n].contiguous()
+                torch.cuda.synchronize()
+                ev[0].record()
+                m.forward(prompt)
+                ev[1].record()
+                tok = ids[:, :1].contiguous()
+                for _ in range(steps):
+                    m.forward(tok)
+                ev[2].record()
+                torch.cuda.synchronize()
+                if rep >= 2:
+                    ts.append(ev[0].elapsed_time(ev[1]))
+                    ds.append(ev[1].elapsed_time(ev[2]) / steps)
+            out[n] = (statistics.median(ts), statistics.median(ds))
+        m.check_status()
+        return out
+
+    entries, qwen_done = [], {}
+    for name, (cfg, qcfg) in lm_sizes().items():
+        if args.only and args.only not in name:
+            continue
+        sampler = ClockSampler(D.local, interval_ms=1000)
+        if not args.no_clock_sampling:
+            sampler.start()
+        m = DuzozenForCausalLM(cfg, max_tokens=8192)
+        m.load_weights(_device_weights(torch, cfg.tensor_shapes()))
+        got = measure(m, cfg.vocab, (512, 4096))
+        m.close()
+        torch.cuda.empty_cache()
+        key = (qcfg.hidden_size, qcfg.num_hidden_layers)
+        if key not in qwen_done and not args.no_closest:
+            q = Q.Qwen3ForCausalLM(qcfg, batch=1)
+            H, I, V = qcfg.hidden_size, qcfg.intermediate_size, qcfg.vocab_size
+            nq, nk = qcfg.num_attention_heads * 128, qcfg.num_key_value_heads * 128
+            rows = {"qkv": (nq + 2 * nk, H), "o": (H, nq), "gate_up": (2 * I, H), "down": (H, I)}
+
+            def bits(shape, seed):
+                g = torch.Generator(device="cuda").manual_seed(seed)
+                t = (torch.randn(shape, generator=g, device="cuda") * 0.02).to(torch.bfloat16)
+                return t.view(torch.int16).cpu().numpy().view("uint16")
+
+            import numpy as np
+            w = {"embed": bits((V, H), 1), "norm": np.ones(H, np.float32)}
+            for l in range(qcfg.num_hidden_layers):
+                for i, (n, shape) in enumerate(rows.items()):
+                    w[(n, l)] = bits(shape, 100 + 4 * l + i)
+                w[("q_norm", l)] = w[("k_norm", l)] = np.ones(128, np.float32)
+                w[("norm1", l)] = w[("norm2", l)] = np.ones(H, np.float32)
+            q.load_weights(w)
+            qwen_done[key] = measure(q, qcfg.vocab_size, (512, 4096))
+            q.close()
+            del w
+            torch.cuda.empty_cache()
+        clocks = sampler.stop() if not args.no_clock_sampling else None
+        W = cfg.width
+        att = sum(W * (x.heads * (x.dim + x.vdim) + x.kv_heads * (x.dim + x.vdim)) for x in cfg.layers)
+        ff = sum(2 * W * x.ff if x.mlp == MLP_DENSE else
+                 x.top * x.experts / (x.experts + x.identity) * 3 * W * x.ff + (x.experts + x.identity) * W
+                 for x in cfg.layers if x.mlp in (MLP_DENSE, MLP_MOE))
+        head = W * cfg.vocab
+
+        def kv_bytes(ctx):
+            return sum(min(ctx, x.window or ctx) * x.kv_heads * (x.dim + x.vdim) * 2 for x in cfg.layers)
+
+        def att_flops(n):  # window-limited causal pairs
+            return sum(2 * x.heads * (x.dim + x.vdim) * (n * min(n, x.window) - min(n, x.window) ** 2 / 2) for x in cfg.layers)
+
+        e = {"metric": "lm_tokens_per_s", "model": "Duzozen", "size": name, "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
+             "data": "synthetic", "repetitions": reps, "clocks": clocks,
+             "config": {"l2": "weights larger than L2; prompts and weights of one size run back to back"}}
+        for n, (pre, dec) in got.items():
+            flops = 2 * n * (att + ff) + att_flops(n) + 2 * head
+            bts = 2 * (att + ff + head) + kv_bytes(n + 64)
+            e[f"prompt_{n}"] = {
+                "prefill_tokens_per_s": n / (pre * 1e-3), "prefill_ms": pre, "prefill_tflops": flops / (pre * 1e-3) / 1e12,
+                "prefill_frac_of_bf16_peak": flops / (pre * 1e-3) / 1e12 / peaks["bf16_tflops"],
+                "decode_tokens_per_s": 1e3 / dec, "decode_ms": dec, "decode_gbs": bts / (dec * 1e-3) / 1e9,
+                "decode_frac_of_copy_bandwidth": bts / (dec * 1e-3) / 1e9 / peaks["hbm_gbs"]}
+        if key in qwen_done:
+            H, I, nl = qcfg.hidden_size, qcfg.intermediate_size, qcfg.num_hidden_layers
+            per = H * 128 * (2 * qcfg.num_attention_heads + 2 * qcfg.num_key_value_heads) + 3 * H * I
+            e["qwen3_equal_size"] = {}
+            for n, (pre, dec) in qwen_done[key].items():
+                flops = 2 * n * per * nl + nl * 2 * qcfg.num_attention_heads * 256 * n * n / 2 + 2 * H * qcfg.vocab_size
+                bts = 2 * (per * nl + H * qcfg.vocab_size) + nl * 2 * qcfg.num_key_value_heads * 128 * 4 * (n + 64)
+                e["qwen3_equal_size"][f"prompt_{n}"] = {
+                    "prefill_tokens_per_s": n / (pre * 1e-3), "prefill_ms": pre,
+                    "prefill_frac_of_bf16_peak": flops / (pre * 1e-3) / 1e12 / peaks["bf16_tflops"],
+                    "decode_tokens_per_s": 1e3 / dec, "decode_ms": dec,
+                    "decode_frac_of_copy_bandwidth": bts / (dec * 1e-3) / 1e9 / peaks["hbm_gbs"]}
+        entries.append(e)
+    D.close()
+    return entries
+
+
 # ======================================================================================= driver of the children
-ARMS = {"attn": attention_arm, "decode": decode_arm, "chain": chain_arm, "gemm32": gemm32_arm,
+ARMS = {"attn": attention_arm, "decode": decode_arm, "chain": chain_arm, "gemm32": gemm32_arm, "lm": lm_arm,
         "gemm_weak": lambda a: gemm_arm(a, weak=True)}
 
 
@@ -865,7 +1024,8 @@ def main() -> None:
     ap.add_argument("--steps", type=int, default=20)
     ap.add_argument("--warmup", type=int, default=3)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="all", choices=["all", "gemm", "gemm_weak", "gemm32", "attn", "chain", "decode"],
+    ap.add_argument("--workload", default="all", choices=["all", "gemm", "gemm_weak", "gemm32", "attn", "chain", "decode",
+                                                               "lm"],
                     help="all (default): the headline GEMM line with the other workloads in its `secondary` array; a "
                          "name: that workload alone, printed as its own line")
     ap.add_argument("--child", default=None, help=argparse.SUPPRESS)
@@ -875,6 +1035,8 @@ def main() -> None:
     ap.add_argument("--no-clock-sampling", action="store_true", help="decode workload: do not run nvidia-smi beside it")
     ap.add_argument("--no-e2e", action="store_true", help="skip the host-buffer leg (profiling captures only)")
     ap.add_argument("--new-tokens", type=int, default=256, help="decode workload: tokens generated per sequence")
+    ap.add_argument("--only", default="", help="lm workload: sizes whose name contains this")
+    ap.add_argument("--no-closest", action="store_true", help="lm workload: leave the Qwen3 decoder out")
     ap.add_argument("--batch", type=int, default=0,
                     help="batch items per rank and step; anything but the default is a profiling case, not a bench line")
     args = ap.parse_args()

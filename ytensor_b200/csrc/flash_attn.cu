@@ -60,6 +60,7 @@ struct FlashParams {
   // ((key_tile0 + j) % ring_tiles) * 128 .., row r sees key c iff r + causal_off - window < c <= r + causal_off
   int window, key_tile0, ring_tiles;
   float cap_log2;            // softcap * log2(e), 0 = scores are not capped
+  float cap_raw;             // scale / softcap: tanh's argument per raw score
   float cap_in;              // 2 * log2(e) * scale / softcap: 2^(raw * cap_in) = exp(2 * scale * raw / softcap)
 };
 
@@ -131,6 +132,26 @@ __device__ __forceinline__ void exp2_emu2(uint64_t x2, float& p0, float& p1) {
   f2_unpack(q2, q0, q1);
   p0 = __int_as_float(__float_as_int(q0) + (__float_as_int(t0) << 23));
   p1 = __int_as_float(__float_as_int(q1) + (__float_as_int(t1) << 23));
+}
+
+__device__ __forceinline__ uint64_t f2_mul(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+// tanh of a packed pair with |y| <= FA_SERIES_MAX: the Taylor series up to y^13 (the next term is 1.5e-3 y^15, 4e-8 at the
+// end of the range).
+constexpr float FA_SERIES_MAX = 0.5f;
+__device__ __forceinline__ uint64_t f2_tanh_series(uint64_t y) {
+  const uint64_t t = f2_mul(y, y);
+  auto k = [](double v) { return f2_pack(static_cast<float>(v), static_cast<float>(v)); };
+  uint64_t q = f2_fma(t, k(21844.0 / 6081075.0), k(-1382.0 / 155925.0));
+  q = f2_fma(q, t, k(62.0 / 2835.0));
+  q = f2_fma(q, t, k(-17.0 / 315.0));
+  q = f2_fma(q, t, k(2.0 / 15.0));
+  q = f2_fma(q, t, k(-1.0 / 3.0));
+  q = f2_mul(q, t);
+  return f2_fma(q, y, y);
 }
 
 // 1 / x by the special-function unit (rcp.approx.ftz, relative error about 2^-23; 1 / inf = 0).
@@ -508,6 +529,43 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
               tmem_ld_32x32b_x64(ts + c0, r);
               tmem_ld_wait();
               const int hi = full ? 64 : cl - c0, lo = full ? 0 : cw - c0;
+              // Small scores (|score| <= softcap / 2 in every row of the warp, the usual case) take tanh from its
+              // Taylor series on the FMA pipe; the general form needs two special-function results per score on top
+              // of the exponential, which that unit would make the bottleneck.
+              bool series = false;
+              if (capped) {
+                float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+                for (int e = 0; e < 64; e += 4) {
+                  a0 = fmax3(a0, fabsf(__uint_as_float(r[e])), fabsf(__uint_as_float(r[e + 1])));
+                  a1 = fmax3(a1, fabsf(__uint_as_float(r[e + 2])), fabsf(__uint_as_float(r[e + 3])));
+                }
+                series = __all_sync(0xffffffffu, fmaxf(a0, a1) * fabsf(p.cap_raw) <= FA_SERIES_MAX);
+              }
+              auto body_series = [&](auto is_limited) {
+                const uint64_t s2 = f2_pack(p.cap_raw, p.cap_raw), c2 = f2_pack(p.cap_log2, p.cap_log2);
+                const uint64_t sh2 = f2_pack(shift - p.cap_log2, shift - p.cap_log2);
+                uint64_t lacc = f2_pack(0.f, 0.f);
+#pragma unroll
+                for (int e = 0; e < 64; e += 2) {
+                  const uint64_t y = f2_mul(f2_pack(__uint_as_float(r[e]), __uint_as_float(r[e + 1])), s2);
+                  const uint64_t x2 = f2_fma(f2_tanh_series(y), c2, sh2);
+                  float t0, t1;
+                  f2_unpack(x2, t0, t1);
+                  t0 = fast_exp2(t0);
+                  t1 = fast_exp2(t1);
+                  if (decltype(is_limited)::value) {
+                    t0 = (e <= hi && e >= lo) ? t0 : 0.f;
+                    t1 = (e + 1 <= hi && e + 1 >= lo) ? t1 : 0.f;
+                  }
+                  lacc = f2_add(lacc, f2_pack(t0, t1));
+                  pk[e >> 1] = pack_bf16x2_rn(t0, t1);
+                }
+                float la, lb;
+                f2_unpack(lacc, la, lb);
+                l0 += la;
+                l1 += lb;
+              };
               auto body = [&](auto is_capped) {
 #pragma unroll
                 for (int e = 0; e < 64; e += 2) {
@@ -526,7 +584,9 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
                   pk[e >> 1] = pack_bf16x2_rn(v[0], v[1]);
                 }
               };
-              if (capped) body(std::true_type{});
+              if (series && full) body_series(std::false_type{});
+              else if (series) body_series(std::true_type{});
+              else if (capped) body(std::true_type{});
               else body(std::false_type{});
             }
             tmem_st_32x32b_x32(ts + (c0 >> 1), pk);
@@ -1658,6 +1718,7 @@ int window_attention(const WindowAttn& a, cudaStream_t st) {
     p.window = a.window > 0 ? a.window : 0x3fffffff;
     p.scale_log2 = a.scale * FA_LOG2E;
     p.cap_log2 = a.softcap > 0.f ? a.softcap * FA_LOG2E : 0.f;
+    p.cap_raw = a.softcap > 0.f ? a.scale / a.softcap : 0.f;
     p.cap_in = a.softcap > 0.f ? 2.f * FA_LOG2E * a.scale / a.softcap : 0.f;
     p.is_bf16 = 1;
     p.pair_heads = (a.groups % 2 == 0) ? 1 : 0;
@@ -1765,7 +1826,7 @@ int ytcuda_flash_attn_fwd(int dtype, const void* Q, const void* K, const void* V
     p.causal = causal; p.causal_off = causal_offset;
     p.scale_log2 = scale * FA_LOG2E;
     p.window = p.key_tile0 = p.ring_tiles = 0;
-    p.cap_log2 = p.cap_in = 0.f;
+    p.cap_log2 = p.cap_raw = p.cap_in = 0.f;
     p.is_bf16 = dtype == YTC_BF16;
     p.pair_heads = (groups % 2 == 0) ? 1 : 0;
     const uint32_t fmt = dtype == YTC_BF16 ? 1u : 0u;
