@@ -1,11 +1,13 @@
 // One new token of a windowed language model: the kernels of a decode step.
 //
 // A step is a chain of short kernels (projection with the norms before it, attention, projection, ...) queued as
-// programmatic dependent launches inside a CUDA graph. Every kernel requests the weights (or the old keys and values) it
-// will multiply by BEFORE it waits for the kernel in front of it, so that the weight stream does not stop at kernel
-// boundaries: two kernels of the chain are resident at a time (256 threads, at most 128 registers). Activations are
-// fp32 vectors of a few KB; every CTA stages the whole vector in shared memory and recomputes the norms from it, which
-// costs less than one more hand-over.
+// programmatic dependent launches inside a CUDA graph. Every kernel requests what does not depend on the kernel in
+// front of it (the weights it will multiply by, norm weights, the residual row, old keys and values) BEFORE it waits for
+// that kernel, so that the weight stream does not stop at kernel boundaries. A kernel lets the next one start once it
+// has passed its own wait: at most two kernels of the chain run at a time, and what a kernel reads before its wait was
+// written at least two kernels earlier. Activations are fp32 vectors of a few KB; every CTA stages the whole vector in
+// shared memory and recomputes the norms from it, which costs less than one more hand-over. Loops are kept rolled:
+// a kernel of this chain runs its code once, at the speed the instructions arrive.
 #include <math_constants.h>
 
 #include "lm_ops.cuh"
@@ -13,15 +15,26 @@
 namespace ytk {
 
 constexpr int DL_THREADS = 256, DL_WARPS = DL_THREADS / 32;
-constexpr int DL_UN = 4;          // row-pair pieces per batch of loads; two batches are in flight
-constexpr int DL_PIECE = 256;     // columns a warp covers with one 16-byte load per lane
+constexpr int DL_PIECE = 256;              // columns a warp covers with one 16-byte load per lane
+constexpr int DL_DEPTH = 8;                // row-pair pieces in flight per warp
+constexpr int DL_RING = DL_DEPTH * 2 * 512;  // bytes of a warp's weight ring
 
-__device__ __forceinline__ uint4 ld_weights(const uint16_t* p) {
-  uint4 v;
-  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0, %1, %2, %3}, [%4];"
-               : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w)
-               : "l"(p));
-  return v;
+// ---------------------------------------------------------------- asynchronous copies of 16 bytes per lane
+__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))),
+               "l"(src)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async16_or_zero(void* dst, const void* src, bool ok) {
+  const int bytes = ok ? 16 : 0;  // (0: the 16 bytes are zero-filled, nothing is read)
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))),
+               "l"(src), "r"(bytes)
+               : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+__device__ __forceinline__ void cp_async_wait() {
+  asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory");
 }
 
 __device__ __forceinline__ float dl_block_sum(float v, float* red) {
@@ -35,123 +48,162 @@ __device__ __forceinline__ float dl_block_sum(float v, float* red) {
   return t;
 }
 
-// Stages the input vector of `k` floats into xs[0 .. padded), zero beyond k. `writer`: this CTA stores the new residual
-// row (and the normed vector, when h_out is given).
-__device__ __forceinline__ void stage_input(const DecodeInput& in, int k, int padded, float* xs, float* red, bool writer,
-                                            float* h_out) {
-  for (int c = k + threadIdx.x; c < padded; c += DL_THREADS) xs[c] = 0.f;
+// ---------------------------------------------------------------- the staged input vector
+// Element c of the vector stands where the lane that multiplies it reads 16 bytes without bank conflicts: a piece of
+// 256 is 32 lanes x 8 elements, first the lanes' elements 0 .. 3, then 4 .. 7.
+__device__ __forceinline__ int staged_at(int c) { return (c & ~255) + ((c & 4) << 5) + ((c & 255) >> 3) * 4 + (c & 3); }
+
+struct InputSmem {  // shared memory of a staged input
+  float* h;         // [padded] the vector, in staged order
+  float *x, *g_post, *g_pre;  // [k] residual row and norm weights (kind 2: unused)
+};
+static int input_floats(int kind, int k, int padded) { return padded + (kind == 2 ? 0 : 3 * k); }
+__device__ __forceinline__ InputSmem input_smem(float* p, int k, int padded) {
+  return InputSmem{p, p + padded, p + padded + k, p + padded + 2 * k};
+}
+
+// Requests what the input needs besides the output of the kernel before (one copy group).
+__device__ __forceinline__ void prefetch_input(const DecodeInput& in, int k, const InputSmem& s) {
+  if (in.kind != 2)
+    for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
+      cp_async16(s.g_pre + c, in.w_pre + c);
+      if (in.kind == 1) {
+        cp_async16(s.g_post + c, in.w_post + c);
+        cp_async16(s.x + c, in.x_in + c);
+      }
+    }
+  cp_async_commit();
+}
+
+// After the wait. `older`: copy groups issued after prefetch_input that may still be in flight. `writer`: this CTA
+// stores the new residual row (and the normed vector, when h_out is given).
+template <int OLDER>
+__device__ __forceinline__ void stage_input(const DecodeInput& in, int k, int padded, const InputSmem& s, float* red,
+                                            bool writer, float* h_out) {
+  for (int c = k + threadIdx.x * 4; c < padded; c += DL_THREADS * 4)
+    *reinterpret_cast<float4*>(s.h + staged_at(c)) = make_float4(0.f, 0.f, 0.f, 0.f);
   if (in.kind == 2) {
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4)
-      *reinterpret_cast<float4*>(xs + c) = *reinterpret_cast<const float4*>(in.plain + c);
+      *reinterpret_cast<float4*>(s.h + staged_at(c)) = *reinterpret_cast<const float4*>(in.plain + c);
     __syncthreads();
     return;
   }
+  float ss = 0.f;
   if (in.kind == 0) {
     int id = *in.id;
     id = id < 0 ? 0 : (id >= in.vocab ? in.vocab - 1 : id);
     const uint16_t* row = in.embed + static_cast<int64_t>(id) * k;
-    for (int c = threadIdx.x; c < k; c += DL_THREADS) {
-      const float v = bf16_bits_to_f32(row[c]);
-      xs[c] = v;
-      if (writer) in.x_out[c] = v;
+    for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
+      const uint2 u = *reinterpret_cast<const uint2*>(row + c);
+      const float4 x = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u),
+                                   __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+      *reinterpret_cast<float4*>(s.x + c) = x;  // (every thread reads back its own columns only)
+      if (writer) *reinterpret_cast<float4*>(in.x_out + c) = x;
     }
+    cp_async_wait<OLDER>();
   } else {
-    float ss = 0.f;
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
       const float4 y = *reinterpret_cast<const float4*>(in.y + c);
-      *reinterpret_cast<float4*>(xs + c) = y;  // (read back by this thread only)
+      *reinterpret_cast<float4*>(s.h + staged_at(c)) = y;
       ss = fmaf(y.x, y.x, ss); ss = fmaf(y.y, y.y, ss); ss = fmaf(y.z, y.z, ss); ss = fmaf(y.w, y.w, ss);
     }
     const float inv = 1.0f / sqrtf(dl_block_sum(ss, red) / in.width + in.eps);
+    cp_async_wait<OLDER>();
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
-      const float4 y = *reinterpret_cast<const float4*>(xs + c), g = *reinterpret_cast<const float4*>(in.w_post + c);
-      float4 x = *reinterpret_cast<const float4*>(in.x_in + c);
+      const float4 y = *reinterpret_cast<const float4*>(s.h + staged_at(c)), g = *reinterpret_cast<const float4*>(s.g_post + c);
+      float4 x = *reinterpret_cast<const float4*>(s.x + c);
       x.x += y.x * inv * g.x; x.y += y.y * inv * g.y; x.z += y.z * inv * g.z; x.w += y.w * inv * g.w;
-      *reinterpret_cast<float4*>(xs + c) = x;
+      *reinterpret_cast<float4*>(s.x + c) = x;
       if (writer) *reinterpret_cast<float4*>(in.x_out + c) = x;
     }
   }
-  __syncthreads();
-  float ss = 0.f;
+  ss = 0.f;
   for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
-    const float4 x = *reinterpret_cast<const float4*>(xs + c);
+    const float4 x = *reinterpret_cast<const float4*>(s.x + c);
     ss = fmaf(x.x, x.x, ss); ss = fmaf(x.y, x.y, ss); ss = fmaf(x.z, x.z, ss); ss = fmaf(x.w, x.w, ss);
   }
   const float inv = 1.0f / sqrtf(dl_block_sum(ss, red + DL_WARPS) / in.width + in.eps);
   for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
-    const float4 g = *reinterpret_cast<const float4*>(in.w_pre + c);
-    float4 x = *reinterpret_cast<const float4*>(xs + c);
+    const float4 g = *reinterpret_cast<const float4*>(s.g_pre + c);
+    float4 x = *reinterpret_cast<const float4*>(s.x + c);
     x.x *= inv * g.x; x.y *= inv * g.y; x.z *= inv * g.z; x.w *= inv * g.w;
-    *reinterpret_cast<float4*>(xs + c) = x;
+    *reinterpret_cast<float4*>(s.h + staged_at(c)) = x;
     if (writer && h_out) *reinterpret_cast<float4*>(h_out + c) = x;
   }
   __syncthreads();
 }
 
-// The product loop. A CTA owns output row pairs [begin, end); KS warps share a pair and split its pieces of 256
-// columns. addr(pair, piece, r): the lane's 16 bytes of weight row 2 pair + r (null beyond the row's end). Partial sums
-// go to part[(pair - begin) * 2 + r][sub].
+// ---------------------------------------------------------------- products of weight rows with the staged vector
+// A CTA owns output row pairs [begin, end); `ks` warps share a pair and split its pieces of 256 columns. Every lane
+// copies its own 16 bytes of both rows of a piece into the warp's ring in shared memory and reads them back itself:
+// DL_DEPTH pieces are in flight, no barrier is involved, and the loop stays rolled. addr(pair, piece, &row0, &row1, &ok)
+// gives the lane's addresses (ok: inside the row). Partial sums go to part[((pair - begin) * 2 + r) * ks + sub].
 template <typename Addr>
 struct RowPairs {
   Addr addr;
-  int end, pieces, ks, sub, slots;
-  int lp, lpc;               // loader's cursor
-  int cp, cpc;               // consumer's cursor
-  float a0 = 0.f, a1 = 0.f;
-  __device__ RowPairs(Addr f, int begin, int end_, int pieces_, int ks_) : addr(f), end(end_), pieces(pieces_), ks(ks_) {
+  uint8_t* ring;
+  int end, pieces, ks, sub, slots, begin;
+  int lp, lpc, ls = 0;  // next piece to request: pair, piece, ring slot
+  __device__ RowPairs(Addr f, uint8_t* rings, int begin_, int end_, int pieces_, int ks_)
+      : addr(f), end(end_), pieces(pieces_), ks(ks_), begin(begin_) {
     const int warp = threadIdx.x >> 5;
+    ring = rings + warp * DL_RING + (threadIdx.x & 31) * 16;
     sub = warp % ks;
     slots = DL_WARPS / ks;
-    lp = cp = begin + warp / ks;
-    lpc = cpc = sub;
-    if (sub >= pieces) lp = cp = end;  // (ks never exceeds the pieces; kept for safety)
+    lp = begin + warp / ks;
+    lpc = sub;
   }
-  __device__ __forceinline__ bool more() const { return cp < end; }
-  __device__ __forceinline__ void load(uint4 (&buf)[DL_UN][2]) {
-#pragma unroll
-    for (int u = 0; u < DL_UN; ++u) {
-      buf[u][0] = buf[u][1] = make_uint4(0u, 0u, 0u, 0u);
-      if (lp >= end) continue;
-      const uint16_t* p0 = addr(lp, lpc, 0);
-      const uint16_t* p1 = addr(lp, lpc, 1);
-      if (p0) buf[u][0] = ld_weights(p0);
-      if (p1) buf[u][1] = ld_weights(p1);
+  __device__ __forceinline__ void request() {  // one copy group, empty past the end
+    if (lp < end) {
+      const uint16_t *p0, *p1;
+      bool ok0, ok1;
+      addr(lp, lpc, p0, p1, ok0, ok1);
+      cp_async16_or_zero(ring + ls * 1024, p0, ok0);
+      cp_async16_or_zero(ring + ls * 1024 + 512, p1, ok1);
       lpc += ks;
       if (lpc >= pieces) {
         lpc = sub;
         lp += slots;
       }
     }
+    cp_async_commit();
+    ls = (ls + 1) & (DL_DEPTH - 1);
   }
-  // xs: the staged vector, piece p at xs + 256 p
-  __device__ __forceinline__ void consume(const uint4 (&buf)[DL_UN][2], const float* xs, float* part, int begin) {
-    const int lane = threadIdx.x & 31;
+  __device__ __forceinline__ void start() {  // DL_DEPTH - 1 groups
+#pragma unroll 1
+    for (int i = 0; i < DL_DEPTH - 1; ++i) request();
+  }
+  // h: the staged vector, piece p at h + 256 p
+  __device__ __forceinline__ void run(const float* h, float* part) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int slot = 0;
+#pragma unroll 1
+    for (int pair = begin + warp / ks; pair < end; pair += slots) {
+      float a0 = 0.f, a1 = 0.f;
+#pragma unroll 1
+      for (int piece = sub; piece < pieces; piece += ks) {
+        request();
+        cp_async_wait<DL_DEPTH - 1>();
+        const uint4 w0 = *reinterpret_cast<const uint4*>(ring + slot * 1024);
+        const uint4 w1 = *reinterpret_cast<const uint4*>(ring + slot * 1024 + 512);
+        slot = (slot + 1) & (DL_DEPTH - 1);
+        const float4 xa = *reinterpret_cast<const float4*>(h + piece * DL_PIECE + lane * 4);
+        const float4 xb = *reinterpret_cast<const float4*>(h + piece * DL_PIECE + 128 + lane * 4);
+        const float x[8] = {xa.x, xa.y, xa.z, xa.w, xb.x, xb.y, xb.z, xb.w};
+        float w[8];
+        Vec8<uint16_t>::unpack(w0, w);
 #pragma unroll
-    for (int u = 0; u < DL_UN; ++u) {
-      if (cp >= end) return;
-      float x[8], w[8];
-      Vec8<float>::load(xs + cpc * DL_PIECE + lane * 8, x);
-      Vec8<uint16_t>::unpack(buf[u][0], w);
+        for (int e = 0; e < 8; ++e) a0 = fmaf(x[e], w[e], a0);
+        Vec8<uint16_t>::unpack(w1, w);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) a0 = fmaf(x[e], w[e], a0);
-      Vec8<uint16_t>::unpack(buf[u][1], w);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) a1 = fmaf(x[e], w[e], a1);
-      cpc += ks;
-      if (cpc >= pieces) {
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-          a0 += __shfl_xor_sync(0xffffffffu, a0, o);
-          a1 += __shfl_xor_sync(0xffffffffu, a1, o);
-        }
-        if (lane == 0) {
-          part[((cp - begin) * 2) * ks + sub] = a0;
-          part[((cp - begin) * 2 + 1) * ks + sub] = a1;
-        }
-        a0 = a1 = 0.f;
-        cpc = sub;
-        cp += slots;
+        for (int e = 0; e < 8; ++e) a1 = fmaf(x[e], w[e], a1);
       }
+      // both sums at once: the lower half of the warp finishes row 0, the upper half row 1
+      const float other = __shfl_xor_sync(0xffffffffu, lane < 16 ? a1 : a0, 16);
+      float v = (lane < 16 ? a0 : a1) + other;
+#pragma unroll
+      for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+      if ((lane & 15) == 0) part[((pair - begin) * 2 + (lane >> 4)) * ks + sub] = v;
     }
   }
 };
@@ -162,7 +214,7 @@ __device__ __forceinline__ float sum_sub(const float* part, int row, int ks) {
   return s;
 }
 
-// Warps that share a row pair: the count with the fewest rounds of pieces per warp.
+// Warps that share a row pair: the count with the fewest pieces per warp.
 static int pick_ks(int pairs_per_cta, int pieces) {
   int best = 1;
   double best_cost = 1e30;
@@ -178,33 +230,46 @@ static int pick_ks(int pairs_per_cta, int pieces) {
   return best;
 }
 
+__device__ __forceinline__ void my_pairs(int pairs, int& begin, int& end) {
+  begin = static_cast<int>(static_cast<int64_t>(pairs) * blockIdx.x / gridDim.x);
+  end = static_cast<int>(static_cast<int64_t>(pairs) * (blockIdx.x + 1) / gridDim.x);
+}
+
+static int dl_smem_check(const void* fn, int smem, const char* what) {
+  if (smem > 220 * 1024) {
+    set_last_error("decode step: %s does not fit shared memory (%d bytes)", what, smem);
+    return YTC_UNSUPPORTED;
+  }
+  return smem > 48 * 1024 ? ensure_dynamic_smem(fn, smem) : YTC_OK;
+}
+static int check_input(const DecodeInput& in, int k) {
+  YTC_REQUIRE(k > 0 && k % 8 == 0 && (in.kind == 2 || in.width <= k), "decode step: bad vector length %d", k);
+  return YTC_OK;
+}
+
 // ------------------------------------------------------------------ linear
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_linear_kernel(const DecodeLinear p, int ks, int padded) {
-  extern __shared__ float dl_smem[];  // xs[padded], part[]
+__global__ void __launch_bounds__(DL_THREADS) decode_linear_kernel(const DecodeLinear p, int ks, int padded) {
+  extern __shared__ __align__(16) uint8_t dl_smem[];  // weight rings, input, part[]
   __shared__ float red[2 * DL_WARPS];
-  float* xs = dl_smem;
-  float* part = dl_smem + padded;
-  const int pairs = (p.n + 1) / 2;
-  const int begin = static_cast<int>(static_cast<int64_t>(pairs) * blockIdx.x / gridDim.x);
-  const int end = static_cast<int>(static_cast<int64_t>(pairs) * (blockIdx.x + 1) / gridDim.x);
+  const InputSmem in = input_smem(reinterpret_cast<float*>(dl_smem + DL_WARPS * DL_RING), p.k, padded);
+  float* part = in.h + padded + (p.in.kind == 2 ? 0 : 3 * p.k);
+  int begin, end;
+  my_pairs((p.n + 1) / 2, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
-  auto addr = [&](int pair, int piece, int r) -> const uint16_t* {
-    const int row = 2 * pair + r, col = piece * DL_PIECE + lane8;
-    return (row < p.n && col < p.k) ? p.w + static_cast<int64_t>(row) * p.k + col : nullptr;
+  auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
+    const int col = piece * DL_PIECE + lane8;
+    ok0 = col < p.k;
+    ok1 = ok0 && 2 * pair + 1 < p.n;
+    p0 = p.w + static_cast<int64_t>(2 * pair) * p.k + (ok0 ? col : 0);
+    p1 = ok1 ? p0 + p.k : p0;
   };
-  RowPairs<decltype(addr)> rp(addr, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
-  uint4 b0[DL_UN][2], b1[DL_UN][2];
-  rp.load(b0);
-  rp.load(b1);
+  RowPairs<decltype(addr)> rp(addr, dl_smem, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
+  prefetch_input(p.in, p.k, in);
+  rp.start();
   dependent_wait();
   dependent_trigger();
-  stage_input(p.in, p.k, padded, xs, red, blockIdx.x == 0, nullptr);
-  while (rp.more()) {
-    rp.consume(b0, xs, part, begin);
-    rp.load(b0);
-    rp.consume(b1, xs, part, begin);
-    rp.load(b1);
-  }
+  stage_input<DL_DEPTH - 1>(p.in, p.k, padded, in, red, blockIdx.x == 0, nullptr);
+  rp.run(in.h, part);
   __syncthreads();
   for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS) {
     const int row = begin * 2 + i;
@@ -215,11 +280,6 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_linear_kernel(const Deco
   if (p.advance && blockIdx.x == 0 && threadIdx.x == 0) *p.advance += 1;
 }
 
-static int check_input(const DecodeInput& in, int k) {
-  YTC_REQUIRE(k > 0 && k % 8 == 0 && (in.kind == 2 || in.width <= k), "decode step: bad vector length %d", k);
-  return YTC_OK;
-}
-
 int decode_linear(const DecodeLinear& a, cudaStream_t st) {
   int s = check_input(a.in, a.k);
   if (s != YTC_OK) return s;
@@ -227,13 +287,8 @@ int decode_linear(const DecodeLinear& a, cudaStream_t st) {
   const int grid = pairs < sm_count() ? pairs : sm_count();
   const int per = (pairs + grid - 1) / grid;
   const int ks = pick_ks(per, pieces);
-  const int smem = (padded + per * 2 * ks) * static_cast<int>(sizeof(float));
-  if (smem > 200 * 1024) {
-    set_last_error("decode step: a projection of %d x %d does not fit shared memory", a.n, a.k);
-    return YTC_UNSUPPORTED;
-  }
-  if (smem > 48 * 1024 && (s = ensure_dynamic_smem(reinterpret_cast<const void*>(decode_linear_kernel), smem)) != YTC_OK)
-    return s;
+  const int smem = DL_WARPS * DL_RING + (input_floats(a.in.kind, a.k, padded) + per * 2 * ks) * static_cast<int>(sizeof(float));
+  if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_linear_kernel), smem, "a projection")) != YTC_OK) return s;
   YTC_CUDA(launch_overlapped(decode_linear_kernel, dim3(grid), dim3(DL_THREADS), smem, st, a, ks, padded));
   count_launch();
   YTC_CUDA(cudaGetLastError());
@@ -241,12 +296,15 @@ int decode_linear(const DecodeLinear& a, cudaStream_t st) {
 }
 
 // ------------------------------------------------------------------ attention
-// One cluster of CTAs per K/V head; the keys of the window are split over its CTAs, each handles all query heads of the
-// group. Per chunk of keys: keys and values in shared memory (the old ones requested before the wait for the projection),
-// eight lanes per key for the scores of all heads, then the value dim across threads. The CTAs' (max, sum, O) meet
-// through distributed shared memory.
+// One cluster of CTAs per K/V head and block of up to four query heads of its group; the keys of the window are split
+// over all warps of the cluster. A warp works on its own: it copies DA_KW keys and values at a time into its part of
+// shared memory (the first ones requested before the wait for the projection), takes the scores with eight lanes per
+// key, and sums the values with the value dim across its lanes. Warps meet through shared memory, CTAs through
+// distributed shared memory.
 constexpr int DA_MAX_CLUSTER = 8;
-constexpr int DA_GB = 4;  // query heads per pass over the values
+constexpr int DA_GB = 4;  // query heads per cluster
+template <typename T>
+constexpr int DA_KW = sizeof(T) == 2 ? 16 : 8;  // keys per step of a warp
 
 __device__ __forceinline__ float ld_cluster(const float* p, uint32_t rank) {
   uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(p)), r;
@@ -259,207 +317,251 @@ __device__ __forceinline__ void cluster_barrier() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(static_cast<uint32_t>(__cvta_generic_to_shared(dst))),
-               "l"(src)
-               : "memory");
+template <typename T>
+__device__ __forceinline__ void load4(const T* p, float (&f)[4]) {
+  if (sizeof(T) == 4) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w;
+  } else {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    f[0] = __uint_as_float(u.x << 16); f[1] = __uint_as_float(u.x & 0xFFFF0000u);
+    f[2] = __uint_as_float(u.y << 16); f[3] = __uint_as_float(u.y & 0xFFFF0000u);
+  }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_attn_kernel(const DecodeAttn p, int chunk, int ncta) {
-  // q[G][dim], o[G][vdim], score[G][chunk], m[G], l[G], red[8][DA_GB][vdim] (floats), then K[chunk][dim + 16 B],
-  // V[chunk][vdim]
-  extern __shared__ __align__(16) float da_smem[];
-  const int G = p.groups, D = p.dim, Dv = p.vdim;
-  float* q_s = da_smem;
-  float* o_s = q_s + G * D;
-  float* sc = o_s + G * Dv;
-  float* m_s = sc + G * chunk;
-  float* l_s = m_s + G;
-  float* red = l_s + G;
-  red = reinterpret_cast<float*>((reinterpret_cast<uintptr_t>(red) + 15) & ~static_cast<uintptr_t>(15));
-  constexpr int PADE = 16 / sizeof(T);
-  const int kld = D + PADE;
-  T* k_s = reinterpret_cast<T*>(red + DL_WARPS * DA_GB * Dv);
-  T* v_s = k_s + chunk * kld;
+// NV: float4 slots of the value dim per lane (1: up to 128, 2: up to 256).
+template <typename T, int NV>
+__global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAttn p, int ncta, int nbuf) {
+  constexpr int KW = DA_KW<T>, GB = DA_GB;
+  // K/V of the warps [warps][nbuf][KW][dim + vdim] (T), q[GB][dim], o[warps][GB][vdim] (merged into o[0])
+  extern __shared__ __align__(16) uint8_t da_smem[];
+  __shared__ float w_s[DL_WARPS][GB][KW], al_s[DL_WARPS][GB], m_s[DL_WARPS][GB], l_s[DL_WARPS][GB], cm[GB], cl[GB];
+  const int D = p.dim, Dv = p.vdim, row_e = D + Dv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int g = blockIdx.x / ncta, rank = blockIdx.x - g * ncta;
+  T* kv_s = reinterpret_cast<T*>(da_smem) + static_cast<size_t>(warp) * nbuf * KW * row_e;
+  float* q_s = reinterpret_cast<float*>(da_smem + static_cast<size_t>(DL_WARPS) * nbuf * KW * row_e * sizeof(T));
+  float* o_s = q_s + GB * D;
+  const int unit = blockIdx.x / ncta, rank = blockIdx.x - unit * ncta;
+  const int blocks = (p.groups + GB - 1) / GB;
+  const int g = unit / blocks, h0 = (unit - g * blocks) * GB;  // K/V head, first query head of the group
+  const int nh = p.groups - h0 < GB ? p.groups - h0 : GB;
 
   // (the position word was written before this step's first kernel started)
   const int pos = *p.pos;
   const int seen = (p.window > 0 && pos + 1 > p.window) ? p.window : pos + 1;
-  const int old_first = pos + 1 - seen, old_n = seen - 1;  // positions old_first .. pos - 1, then the new one
-  const int per = (old_n + ncta - 1) / ncta;
-  int k0 = rank * per;
-  int k1 = k0 + per < old_n ? k0 + per : old_n;
-  if (k0 > k1) k0 = k1;
-  const int mine = k1 - k0 + (rank == 0 ? 1 : 0);  // CTA 0 also takes the new key, after its old ones
+  const int old_n = seen - 1;  // positions pos - old_n .. pos - 1, then the new one
+  const int warps = ncta * DL_WARPS, wi = rank * DL_WARPS + warp;
+  const int per = (old_n + warps - 1) / warps;
+  const int k0 = wi * per < old_n ? wi * per : old_n;
+  const int k1 = k0 + per < old_n ? k0 + per : old_n;
+  const bool has_new = wi == warps - 1;  // the last warp (the one with the fewest old keys) takes the new key
+  const int mine = k1 - k0 + (has_new ? 1 : 0);
   const T* kr = static_cast<const T*>(p.k) + static_cast<int64_t>(g) * p.ring * D;
   const T* vr = static_cast<const T*>(p.v) + static_cast<int64_t>(g) * p.ring * Dv;
+  const int row0 = (pos - old_n + k0) % p.ring;
   constexpr int VE = 16 / sizeof(T);  // elements per 16 bytes
-  auto fetch = [&](int c0) {  // requests old keys c0 .. of this CTA
-    const int n_old = (k1 - k0) - c0 < chunk ? (k1 - k0) - c0 : chunk;
-    const int kp = D / VE, vp = Dv / VE;
-    for (int i = threadIdx.x; i < n_old * (kp + vp); i += DL_THREADS) {
-      const int key = i / (kp + vp), c = i - key * (kp + vp);
-      const int64_t row = (old_first + k0 + c0 + key) % p.ring;
-      if (c < kp) cp_async16(k_s + key * kld + c * VE, kr + row * D + c * VE);
-      else cp_async16(v_s + key * Dv + (c - kp) * VE, vr + row * Dv + (c - kp) * VE);
+  const int kp = D / VE, vp = Dv / VE;
+  auto fetch = [&](int c0, int buf) {  // requests old keys c0 .. of this warp (one copy group)
+    T* dst = kv_s + buf * KW * row_e;
+    const int n = (k1 - k0) - c0 < KW ? (k1 - k0) - c0 : KW;
+    int row = row0 + c0;
+#pragma unroll 1
+    for (int key = 0; key < n; ++key, ++row) {
+      const int64_t r = row >= p.ring ? row - p.ring : row;
+      for (int c = lane; c < kp + vp; c += 32)
+        cp_async16(dst + key * row_e + c * VE, c < kp ? kr + r * D + c * VE : vr + r * Dv + (c - kp) * VE);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    cp_async_commit();
   };
-  fetch(0);
+  fetch(0, 0);
+  if (nbuf > 1) fetch(KW, 1);
   dependent_wait();
   dependent_trigger();
-  const int H = p.kv_heads * G;
-  for (int i = threadIdx.x; i < G * D; i += DL_THREADS) q_s[i] = p.qkv[static_cast<int64_t>(g) * G * D + i];
-  for (int i = threadIdx.x; i < G * Dv; i += DL_THREADS) o_s[i] = 0.f;
-  if (threadIdx.x < G) {
-    m_s[threadIdx.x] = -CUDART_INF_F;
-    l_s[threadIdx.x] = 0.f;
-  }
-  const float* k_new = p.qkv + static_cast<int64_t>(H) * D + static_cast<int64_t>(g) * D;
-  const float* v_new = p.qkv + static_cast<int64_t>(H + p.kv_heads) * D + static_cast<int64_t>(g) * Dv;
-  const float lam = p.mix == VMIX_MIX ? *p.lambda : 0.f;
-  int npv = 1;  // lanes per value row (a power of two), 8 elements each
-  while (npv * 8 < Dv) npv <<= 1;
-  const int piece = threadIdx.x % npv, key_lane = threadIdx.x / npv, key_lanes = DL_THREADS / npv;
-
-  for (int c0 = 0; c0 < mine; c0 += chunk) {
-    const int n = mine - c0 < chunk ? mine - c0 : chunk;
-    if (c0 > 0) {
-      __syncthreads();  // everyone is done with the previous chunk
-      fetch(c0);
-    }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    if (rank == 0 && c0 + n == mine) {  // the new key and value: into the chunk and into the rings
-      const int at = n - 1;
-      const int64_t row = pos % p.ring;
-      T* kw = static_cast<T*>(p.k) + (static_cast<int64_t>(g) * p.ring + row) * D;
-      T* vw = static_cast<T*>(p.v) + (static_cast<int64_t>(g) * p.ring + row) * Dv;
-      for (int i = threadIdx.x; i < (D + Dv) / 8; i += DL_THREADS) {
-        float f[8];
-        if (i < D / 8) {
-          Vec8<float>::load(k_new + i * 8, f);
-          Vec8<T>::store(kw + i * 8, f);
-          Vec8<T>::store(k_s + at * kld + i * 8, f);
-        } else {
-          const int e = i * 8 - D;
-          Vec8<float>::load(v_new + e, f);
-          float* first = p.v_first + static_cast<int64_t>(g) * Dv + e;
-          if (p.mix == VMIX_FIRST) Vec8<float>::store(first, f);
-          if (p.mix == VMIX_MIX) {
-            float v0[8];
-            Vec8<float>::load(first, v0);
+  const int H = p.kv_heads * p.groups;
+  for (int i = threadIdx.x * 4; i < nh * D; i += DL_THREADS * 4)
+    *reinterpret_cast<float4*>(q_s + i) =
+        *reinterpret_cast<const float4*>(p.qkv + static_cast<int64_t>(g * p.groups + h0) * D + i);
+  if (has_new) {  // the new key and value: behind the warp's old keys, and (one cluster per K/V head) into the rings
+    const float* k_new = p.qkv + static_cast<int64_t>(H) * D + static_cast<int64_t>(g) * D;
+    const float* v_new = p.qkv + static_cast<int64_t>(H + p.kv_heads) * D + static_cast<int64_t>(g) * Dv;
+    const float lam = p.mix == VMIX_MIX ? *p.lambda : 0.f;
+    const int64_t row = pos % p.ring;
+    T* kw = static_cast<T*>(p.k) + (static_cast<int64_t>(g) * p.ring + row) * D;
+    T* vw = static_cast<T*>(p.v) + (static_cast<int64_t>(g) * p.ring + row) * Dv;
+    const bool first_block = h0 == 0;
+    for (int i = lane; i < (D + Dv) / 8; i += 32) {
+      float f[8];
+      const int e = i * 8;
+      if (e < D) {
+        Vec8<float>::load(k_new + e, f);
+      } else {
+        Vec8<float>::load(v_new + e - D, f);
+        float* first = p.v_first + static_cast<int64_t>(g) * Dv + e - D;
+        if (p.mix == VMIX_FIRST && first_block) Vec8<float>::store(first, f);
+        if (p.mix == VMIX_MIX) {
+          float v0[8];
+          Vec8<float>::load(first, v0);
 #pragma unroll
-            for (int k = 0; k < 8; ++k) f[k] = (1.f - lam) * f[k] + lam * v0[k];
-          }
-          Vec8<T>::store(vw + e, f);
-          Vec8<T>::store(v_s + at * Dv + e, f);
+          for (int k = 0; k < 8; ++k) f[k] = (1.f - lam) * f[k] + lam * v0[k];
         }
       }
+      if (first_block) Vec8<T>::store(e < D ? kw + e : vw + e - D, f);
+      Vec8<float>::store(o_s + e, f);  // joins the keys in shared memory when their last step is reached
     }
-    __syncthreads();
-    // scores: eight lanes per key
-    for (int key0 = warp * 4; key0 < n; key0 += DL_WARPS * 4) {
+  }
+  __syncthreads();
+  float acc[GB][NV * 4] = {};
+  if (lane < GB) {
+    m_s[warp][lane] = -CUDART_INF_F;
+    l_s[warp][lane] = 0.f;
+  }
+  __syncwarp();
+#pragma unroll 1
+  for (int c0 = 0, buf = 0; c0 < mine; c0 += KW, buf = (buf + 1 == nbuf ? 0 : buf + 1)) {
+    const int n = mine - c0 < KW ? mine - c0 : KW;
+    if (nbuf > 1) cp_async_wait<1>();
+    else cp_async_wait<0>();
+    T* kv = kv_s + buf * KW * row_e;
+    if (has_new && c0 + n == mine) {
+      for (int i = lane; i < row_e / 8; i += 32) {
+        float f[8];
+        Vec8<float>::load(o_s + i * 8, f);
+        Vec8<T>::store(kv + (n - 1) * row_e + i * 8, f);
+      }
+    }
+    __syncwarp();
+    // scores: eight lanes per key, four keys at a time
+#pragma unroll 1
+    for (int key0 = 0; key0 < n; key0 += 4) {
       const int key = key0 + (lane >> 3);
-      const T* kv = k_s + (key < n ? key : 0) * kld;
-      for (int h = 0; h < G; ++h) {
-        float dot = 0.f;
-        for (int c = (lane & 7) * 8; c < D; c += 64) {
-          float a[8], b[8];
-          Vec8<T>::load(kv + c, a);
+      const T* k = kv + (key < n ? key : 0) * row_e;
+      float dot[GB] = {};
+      for (int c = (lane & 7) * 8; c < D; c += 64) {
+        float a[8];
+        Vec8<T>::load(k + c, a);
+#pragma unroll
+        for (int h = 0; h < GB; ++h) {
+          if (h >= nh) break;
+          float b[8];
           Vec8<float>::load(q_s + h * D + c, b);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) dot = fmaf(a[e], b[e], dot);
-        }
-        dot += __shfl_xor_sync(0xffffffffu, dot, 1);
-        dot += __shfl_xor_sync(0xffffffffu, dot, 2);
-        dot += __shfl_xor_sync(0xffffffffu, dot, 4);
-        if ((lane & 7) == 0 && key < n) {
-          dot *= p.scale;
-          sc[h * chunk + key] = p.softcap > 0.f ? p.softcap * tanhf(dot / p.softcap) : dot;
+          for (int e = 0; e < 8; ++e) dot[h] = fmaf(a[e], b[e], dot[h]);
         }
       }
-    }
-    __syncthreads();
-    for (int h = warp; h < G; h += DL_WARPS) {  // weights of a head: one warp
-      float m = -CUDART_INF_F;
-      for (int i = lane; i < n; i += 32) m = fmaxf(m, sc[h * chunk + i]);
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-      const float m_old = m_s[h], m_new = fmaxf(m_old, m);
-      const float alpha = m_old == -CUDART_INF_F ? 0.f : expf(m_old - m_new);
-      float l = 0.f;
-      for (int i = lane; i < n; i += 32) {
-        const float w = expf(sc[h * chunk + i] - m_new);
-        sc[h * chunk + i] = w;
-        l += w;
-      }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-      for (int i = lane; i < Dv; i += 32) o_s[h * Dv + i] *= alpha;
-      __syncwarp();
-      if (lane == 0) {
-        m_s[h] = m_new;
-        l_s[h] = l_s[h] * alpha + l;
+      for (int h = 0; h < GB; ++h) {
+        if (h >= nh) break;
+        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 1);
+        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 2);
+        dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 4);
+        if ((lane & 7) == 0 && key < n) w_s[warp][h][key] = dot[h] * p.scale;
       }
     }
-    __syncthreads();
-    for (int h0 = 0; h0 < G; h0 += DA_GB) {
-      float acc[DA_GB][8] = {};
-      if (piece * 8 < Dv)
-        for (int key = key_lane; key < n; key += key_lanes) {
-          float v[8];
-          Vec8<T>::load(v_s + key * Dv + piece * 8, v);
-#pragma unroll
-          for (int hh = 0; hh < DA_GB; ++hh) {
-            const float w = h0 + hh < G ? sc[(h0 + hh) * chunk + key] : 0.f;
-#pragma unroll
-            for (int e = 0; e < 8; ++e) acc[hh][e] = fmaf(w, v[e], acc[hh][e]);
-          }
-        }
-      for (int o = npv; o < 32; o <<= 1)
-#pragma unroll
-        for (int hh = 0; hh < DA_GB; ++hh)
-#pragma unroll
-          for (int e = 0; e < 8; ++e) acc[hh][e] += __shfl_xor_sync(0xffffffffu, acc[hh][e], o);
-      if (lane < npv && piece * 8 < Dv)
-#pragma unroll
-        for (int hh = 0; hh < DA_GB; ++hh) Vec8<float>::store(red + (warp * DA_GB + hh) * Dv + piece * 8, acc[hh]);
-      __syncthreads();
-      for (int i = threadIdx.x; i < DA_GB * Dv; i += DL_THREADS) {
-        const int hh = i / Dv;
-        if (h0 + hh >= G) break;
-        float s = 0.f;
-#pragma unroll
-        for (int w = 0; w < DL_WARPS; ++w) s += red[w * DA_GB * Dv + i];
-        o_s[h0 * Dv + i] += s;
+    __syncwarp();
+    // weights: KW lanes per head
+#pragma unroll 1
+    for (int h = lane / KW; h < GB; h += 32 / KW) {
+      const int key = lane % KW;
+      float s = -CUDART_INF_F;
+      if (h < nh && key < n) {
+        s = w_s[warp][h][key];
+        if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
       }
-      __syncthreads();
+      float m = s;
+#pragma unroll
+      for (int o = KW / 2; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      const float m_old = m_s[warp][h], m_new = fmaxf(m_old, m);
+      const float w = s == -CUDART_INF_F ? 0.f : expf(s - m_new);
+      float l = w;
+#pragma unroll
+      for (int o = KW / 2; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+      w_s[warp][h][key] = w;
+      if (key == 0) {
+        const float alpha = m_old == -CUDART_INF_F ? 0.f : expf(m_old - m_new);
+        al_s[warp][h] = alpha;
+        m_s[warp][h] = m_new;
+        l_s[warp][h] = l_s[warp][h] * alpha + l;
+      }
     }
+    __syncwarp();
+#pragma unroll
+    for (int h = 0; h < GB; ++h) {
+      const float alpha = al_s[warp][h];
+#pragma unroll
+      for (int e = 0; e < NV * 4; ++e) acc[h][e] *= alpha;
+    }
+#pragma unroll 2
+    for (int key = 0; key < n; ++key) {
+      float v[NV][4] = {};
+#pragma unroll
+      for (int j = 0; j < NV; ++j)
+        if (j * 128 + lane * 4 < Dv) load4<T>(kv + key * row_e + D + j * 128 + lane * 4, v[j]);
+#pragma unroll
+      for (int h = 0; h < GB; ++h) {
+        const float w = w_s[warp][h][key];
+#pragma unroll
+        for (int e = 0; e < NV * 4; ++e) acc[h][e] = fmaf(w, v[e >> 2][e & 3], acc[h][e]);
+      }
+    }
+    __syncwarp();
+    if (c0 + nbuf * KW < mine) fetch(c0 + nbuf * KW, buf);
+    else cp_async_commit();
   }
-  // the cluster's partial results: each CTA finishes a share of the outputs
-  if (ncta > 1) cluster_barrier();
-  else __syncthreads();
-  for (int i = rank * DL_THREADS + threadIdx.x; i < G * Dv; i += ncta * DL_THREADS) {
+  __syncthreads();  // (the new key's copy in o_s has been read)
+#pragma unroll
+  for (int h = 0; h < GB; ++h)
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+      if (j * 128 + lane * 4 < Dv)
+        *reinterpret_cast<float4*>(o_s + (warp * GB + h) * Dv + j * 128 + lane * 4) =
+            make_float4(acc[h][4 * j], acc[h][4 * j + 1], acc[h][4 * j + 2], acc[h][4 * j + 3]);
+  __syncthreads();
+  // the CTA's result, then the cluster's: each CTA finishes a share of the outputs
+  for (int i = threadIdx.x; i < nh * Dv; i += DL_THREADS) {
     const int h = i / Dv;
     float m = -CUDART_INF_F;
-    float ms[DA_MAX_CLUSTER];
+#pragma unroll
+    for (int w = 0; w < DL_WARPS; ++w) m = fmaxf(m, m_s[w][h]);
+    float l = 0.f, o = 0.f;
+#pragma unroll
+    for (int w = 0; w < DL_WARPS; ++w) {
+      const float f = m_s[w][h] == -CUDART_INF_F ? 0.f : expf(m_s[w][h] - m);
+      l = fmaf(f, l_s[w][h], l);
+      o = fmaf(f, o_s[w * GB * Dv + i], o);
+    }
+    o_s[i] = o;  // (the element of warp 0 that this thread alone has read)
+    if (i == h * Dv) {
+      cm[h] = m;
+      cl[h] = l;
+    }
+  }
+  if (ncta > 1) cluster_barrier();
+  else __syncthreads();
+  float* out = p.out + static_cast<int64_t>(g * p.groups + h0) * Dv;
+  for (int i = rank * DL_THREADS + threadIdx.x; i < nh * Dv; i += ncta * DL_THREADS) {
+    const int h = i / Dv;
+    if (ncta == 1) {
+      out[i] = o_s[i] / cl[h];
+      continue;
+    }
+    float ms[DA_MAX_CLUSTER], ls[DA_MAX_CLUSTER], os[DA_MAX_CLUSTER], m = -CUDART_INF_F;
 #pragma unroll
     for (int r = 0; r < DA_MAX_CLUSTER; ++r) {
-      ms[r] = r < ncta ? (ncta > 1 ? ld_cluster(m_s + h, r) : m_s[h]) : -CUDART_INF_F;
+      const uint32_t from = r < ncta ? r : 0;
+      ms[r] = ld_cluster(cm + h, from);
+      ls[r] = ld_cluster(cl + h, from);
+      os[r] = ld_cluster(o_s + i, from);
+      if (r >= ncta) ms[r] = -CUDART_INF_F;
       m = fmaxf(m, ms[r]);
     }
     float l = 0.f, o = 0.f;
 #pragma unroll
     for (int r = 0; r < DA_MAX_CLUSTER; ++r) {
-      if (r >= ncta || ms[r] == -CUDART_INF_F) continue;
-      const float f = expf(ms[r] - m);
-      l += f * (ncta > 1 ? ld_cluster(l_s + h, r) : l_s[h]);
-      o += f * (ncta > 1 ? ld_cluster(o_s + i, r) : o_s[i]);
+      const float f = ms[r] == -CUDART_INF_F ? 0.f : expf(ms[r] - m);
+      l = fmaf(f, ls[r], l);
+      o = fmaf(f, os[r], o);
     }
-    p.out[static_cast<int64_t>(g) * G * Dv + i] = o / l;
+    out[i] = o / l;
   }
   if (ncta > 1) cluster_barrier();  // no CTA leaves while another may still read its shared memory
 }
@@ -486,24 +588,22 @@ static cudaError_t launch_cluster(void (*kernel)(KArgs...), int grid, int cluste
 
 template <typename T>
 static int decode_attention_t(const DecodeAttn& a, cudaStream_t st) {
+  constexpr int KW = DA_KW<T>;
+  const int units = a.kv_heads * ((a.groups + DA_GB - 1) / DA_GB);
   int ncta = 1;
-  while (ncta < DA_MAX_CLUSTER && static_cast<int64_t>(ncta) * 32 < a.max_keys && a.kv_heads * ncta * 2 <= sm_count()) ncta *= 2;
-  const int64_t mine = (a.max_keys + ncta - 1) / ncta + 1;
-  auto bytes = [&](int chunk) {
-    const size_t fl = static_cast<size_t>(a.groups) * (a.dim + a.vdim + chunk + 2) + DL_WARPS * DA_GB * a.vdim + 8;
-    return fl * 4 + static_cast<size_t>(chunk) * (a.dim + 16 / sizeof(T) + a.vdim) * sizeof(T) + 32;
-  };
-  int chunk = static_cast<int>(mine < 256 ? (mine + 7) / 8 * 8 : 256);
-  while (chunk > 8 && bytes(chunk) > 100 * 1024) chunk -= 8;  // two kernels of the chain share an SM
-  if (bytes(chunk) > 220 * 1024) {
-    set_last_error("decode step: %d query heads of %d + %d channels per K/V head do not fit shared memory", a.groups, a.dim,
-                   a.vdim);
-    return YTC_UNSUPPORTED;
-  }
-  const int smem = static_cast<int>(bytes(chunk));
-  const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(decode_attn_kernel<T>), smem);
+  while (ncta < DA_MAX_CLUSTER && static_cast<int64_t>(ncta) * DL_WARPS * 4 < a.max_keys && units * ncta * 2 <= sm_count())
+    ncta *= 2;
+  const int64_t per_warp = (a.max_keys + ncta * DL_WARPS - 1) / (ncta * DL_WARPS) + 1;
+  const int step = DL_WARPS * KW * (a.dim + a.vdim) * static_cast<int>(sizeof(T));
+  // (the new key and value pass through the output area on their way)
+  const int outs = DL_WARPS * DA_GB * a.vdim > a.dim + a.vdim ? DL_WARPS * DA_GB * a.vdim : a.dim + a.vdim;
+  const int rest = (DA_GB * a.dim + outs) * 4;
+  const int nbuf = (per_warp > KW && 2 * step + rest <= 150 * 1024) ? 2 : 1;
+  const int smem = nbuf * step + rest;
+  auto* fn = a.vdim <= 128 ? decode_attn_kernel<T, 1> : decode_attn_kernel<T, 2>;
+  const int s = dl_smem_check(reinterpret_cast<const void*>(fn), smem, "attention");
   if (s != YTC_OK) return s;
-  YTC_CUDA(launch_cluster(decode_attn_kernel<T>, a.kv_heads * ncta, ncta, smem, st, a, chunk, ncta));
+  YTC_CUDA(launch_cluster(fn, units * ncta, ncta, smem, st, a, ncta, nbuf));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
@@ -518,43 +618,51 @@ int decode_attention(const DecodeAttn& a, cudaStream_t st) {
 // ------------------------------------------------------------------ router
 // One cluster: every CTA computes a share of the logits, CTA 0 collects them and routes.
 constexpr int DR_CLUSTER = 8;
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const DecodeRoute p, int padded) {
-  extern __shared__ float dr_smem[];  // xs[padded], scores[n], choice scores[n]
+template <int VPL>
+__global__ void __launch_bounds__(DL_THREADS) decode_route_kernel(const DecodeRoute p, int ks, int padded) {
+  extern __shared__ __align__(16) uint8_t dr_smem[];  // weight rings, input, part[], scores[n], choice scores[n]
   __shared__ float red[2 * DL_WARPS];
-  const int n = p.r.experts + p.r.identity;
-  float* xs = dr_smem;
-  float* s = dr_smem + padded;
+  const int n = p.r.experts + p.r.identity, pairs = (n + 1) / 2;
+  const InputSmem in = input_smem(reinterpret_cast<float*>(dr_smem + DL_WARPS * DL_RING), p.k, padded);
+  float* part = in.h + padded + 3 * p.k;
+  float* s = part + ((pairs + DR_CLUSTER - 1) / DR_CLUSTER) * 2 * ks;
   float* c = s + n;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int rank = blockIdx.x;
+  int begin, end;
+  my_pairs(pairs, begin, end);
+  auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
+    const int col = piece * DL_PIECE + lane * 8;
+    ok0 = col < p.k;
+    ok1 = ok0 && 2 * pair + 1 < n;
+    p0 = p.w + static_cast<int64_t>(2 * pair) * p.k + (ok0 ? col : 0);
+    p1 = ok1 ? p0 + p.k : p0;
+  };
+  RowPairs<decltype(addr)> rp(addr, dr_smem, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
+  prefetch_input(p.in, p.k, in);
+  rp.start();
+  if (rank == 0)  // (brings the correction into the L1 / L2 ahead of its use)
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) c[i] = p.correction[i];
   dependent_wait();
   dependent_trigger();
-  stage_input(p.in, p.k, padded, xs, red, rank == 0, p.h);
-  for (int e = rank * DL_WARPS + warp; e < n; e += DR_CLUSTER * DL_WARPS) {
-    const uint16_t* w = p.w + static_cast<int64_t>(e) * p.k;
-    float acc = 0.f;
-    for (int col = lane * 8; col < p.k; col += DL_PIECE) {
-      float a[8], x[8];
-      Vec8<uint16_t>::load(w + col, a);
-      Vec8<float>::load(xs + col, x);
-#pragma unroll
-      for (int k = 0; k < 8; ++k) acc = fmaf(a[k], x[k], acc);
-    }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) acc += __shfl_xor_sync(0xffffffffu, acc, o);
-    if (lane == 0) s[e] = acc;
-  }
+  stage_input<DL_DEPTH - 1>(p.in, p.k, padded, in, red, rank == 0, p.h);
+  rp.run(in.h, part);
+  __syncthreads();
+  for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS)
+    if (begin * 2 + i < n) s[begin * 2 + i] = sum_sub(part, i, ks);
   cluster_barrier();
   if (rank == 0) {
     for (int e = threadIdx.x; e < n; e += DL_THREADS) {
-      const uint32_t owner = (e / DL_WARPS) % DR_CLUSTER;
+      const int pair = e / 2;
+      int owner = 0;
+      while (pair >= static_cast<int>(static_cast<int64_t>(pairs) * (owner + 1) / DR_CLUSTER)) ++owner;
       if (owner != 0) s[e] = ld_cluster(s + e, owner);
     }
     __syncthreads();
     if (warp == 0) {
       int choice;
       float weight;
-      warp_route(s, c, p.correction, p.r, lane, choice, weight);
+      warp_route<VPL>(s, c, p.correction, p.r, lane, choice, weight);
       if (lane < p.r.top) {
         p.choice[lane] = choice;
         p.weight[lane] = weight;
@@ -567,12 +675,15 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const Decod
 int decode_route(const DecodeRoute& a, cudaStream_t st) {
   int s = check_input(a.in, a.k);
   if (s != YTC_OK) return s;
-  const int n = a.r.experts + a.r.identity;
-  const int padded = (a.k + DL_PIECE - 1) / DL_PIECE * DL_PIECE;
-  const int smem = (padded + 2 * n) * static_cast<int>(sizeof(float));
-  if (smem > 48 * 1024 && (s = ensure_dynamic_smem(reinterpret_cast<const void*>(decode_route_kernel), smem)) != YTC_OK)
-    return s;
-  YTC_CUDA(launch_cluster(decode_route_kernel, DR_CLUSTER, DR_CLUSTER, smem, st, a, padded));
+  const int n = a.r.experts + a.r.identity, pairs = (n + 1) / 2, per = (pairs + DR_CLUSTER - 1) / DR_CLUSTER;
+  const int pieces = (a.k + DL_PIECE - 1) / DL_PIECE, padded = pieces * DL_PIECE;
+  const int ks = pick_ks(per, pieces);
+  const int smem = DL_WARPS * DL_RING +
+                   (input_floats(a.in.kind, a.k, padded) + per * 2 * ks + 2 * n) * static_cast<int>(sizeof(float));
+  auto* fn = n <= 128 ? decode_route_kernel<4> : n <= 256 ? decode_route_kernel<8> : decode_route_kernel<LM_MAX_ROUTES / 32>;
+  YTC_REQUIRE(a.in.kind != 2, "decode step: the router's input is a normed residual row");
+  if ((s = dl_smem_check(reinterpret_cast<const void*>(fn), smem, "the router")) != YTC_OK) return s;
+  YTC_CUDA(launch_cluster(fn, DR_CLUSTER, DR_CLUSTER, smem, st, a, ks, padded));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
@@ -587,56 +698,54 @@ struct Chosen {
   float identity;  // sum of the identity experts' weights
 };
 __device__ __forceinline__ void read_choice(const DecodeExperts& p, Chosen* c) {
-  if (threadIdx.x == 0) {
-    int n = 0;
-    float id = 0.f;
-    for (int k = 0; k < p.r.top; ++k) {
-      const int e = p.choice[k];
-      const float w = p.weight[k];
-      if (e >= p.r.experts) id += w;
-      else if (e >= 0) {
-        c->expert[n] = e;
-        c->slot[n] = k;
-        c->weight[n++] = w;
-      }
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    const int e = lane < p.r.top ? p.choice[lane] : -1;
+    const float w = lane < p.r.top ? p.weight[lane] : 0.f;
+    const bool real = e >= 0 && e < p.r.experts;
+    const uint32_t mask = __ballot_sync(0xffffffffu, real);
+    if (real) {
+      const int i = __popc(mask & ((1u << lane) - 1u));
+      c->expert[i] = e;
+      c->slot[i] = lane;
+      c->weight[i] = w;
     }
-    c->n = n;
-    c->identity = id;
+    float id = e >= p.r.experts ? w : 0.f;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) id += __shfl_xor_sync(0xffffffffu, id, o);
+    if (lane == 0) {
+      c->n = __popc(mask);
+      c->identity = id;
+    }
   }
   __syncthreads();
 }
 
 // act[slot][j] = silu(gate_j . h) * (up_j . h): a row pair is (gate_j, up_j) of one chosen expert
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const DecodeExperts p, int ks, int padded) {
-  extern __shared__ float dg_smem[];
+__global__ void __launch_bounds__(DL_THREADS) decode_gate_up_kernel(const DecodeExperts p, int ks, int padded) {
+  extern __shared__ __align__(16) uint8_t dg_smem[];  // weight rings, input, part[]
   __shared__ Chosen ch;
-  float* xs = dg_smem;
-  float* part = dg_smem + padded;
+  float* xs = reinterpret_cast<float*>(dg_smem + DL_WARPS * DL_RING);
+  float* part = xs + padded;
   dependent_wait();
   dependent_trigger();
   read_choice(p, &ch);
-  const int pairs = ch.n * p.ff;
-  const int begin = static_cast<int>(static_cast<int64_t>(pairs) * blockIdx.x / gridDim.x);
-  const int end = static_cast<int>(static_cast<int64_t>(pairs) * (blockIdx.x + 1) / gridDim.x);
+  int begin, end;
+  my_pairs(ch.n * p.ff, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
-  auto addr = [&](int pair, int piece, int r) -> const uint16_t* {
-    const int col = piece * DL_PIECE + lane8;
-    if (col >= p.k) return nullptr;
-    const int i = pair / p.ff, j = pair - i * p.ff;
-    return p.gate_up + (static_cast<int64_t>(ch.expert[i]) * 2 * p.ff + 2 * j + r) * p.k + col;
+  auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
+    const int col = piece * DL_PIECE + lane8, i = pair / p.ff, j = pair - i * p.ff;
+    ok0 = ok1 = col < p.k;
+    p0 = p.gate_up + (static_cast<int64_t>(ch.expert[i]) * 2 * p.ff + 2 * j) * p.k + (ok0 ? col : 0);
+    p1 = p0 + p.k;
   };
-  RowPairs<decltype(addr)> rp(addr, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
-  uint4 b0[DL_UN][2], b1[DL_UN][2];
-  rp.load(b0);
-  rp.load(b1);
-  for (int c = threadIdx.x; c < padded; c += DL_THREADS) xs[c] = c < p.k ? p.h[c] : 0.f;
+  RowPairs<decltype(addr)> rp(addr, dg_smem, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
+  rp.start();
+  for (int c = threadIdx.x * 4; c < padded; c += DL_THREADS * 4)
+    *reinterpret_cast<float4*>(xs + staged_at(c)) =
+        c < p.k ? *reinterpret_cast<const float4*>(p.h + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   __syncthreads();
-  while (rp.more()) {
-    rp.consume(b0, xs, part, begin);
-    rp.load(b0);
-    rp.consume(b1, xs, part, begin);
-    rp.load(b1);
-  }
+  rp.run(xs, part);
   __syncthreads();
   for (int i = threadIdx.x; i < end - begin; i += DL_THREADS) {
     const int pair = begin + i, e = pair / p.ff, j = pair - e * p.ff;
@@ -646,41 +755,39 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const Dec
 
 // out[n] = sum over the chosen experts of weight * (down_n . act) + (identity weights) * h[n]: the experts' vectors,
 // already multiplied by their weights, stand one after the other in shared memory
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded) {
-  extern __shared__ float dd_smem[];
+__global__ void __launch_bounds__(DL_THREADS) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded) {
+  extern __shared__ __align__(16) uint8_t dd_smem[];  // weight rings, inputs [top][ff_padded], part[]
   __shared__ Chosen ch;
-  float* xs = dd_smem;                            // [top][ff_padded]
-  float* part = dd_smem + p.r.top * ff_padded;
+  float* xs = reinterpret_cast<float*>(dd_smem + DL_WARPS * DL_RING);
+  float* part = xs + p.r.top * ff_padded;
   // (the choice was made two kernels ago: the kernel before this one has already waited for it)
   read_choice(p, &ch);
-  const int pairs = p.k / 2;
-  const int begin = static_cast<int>(static_cast<int64_t>(pairs) * blockIdx.x / gridDim.x);
-  const int end = static_cast<int>(static_cast<int64_t>(pairs) * (blockIdx.x + 1) / gridDim.x);
+  int begin, end;
+  my_pairs(p.k / 2, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
   const int per_expert = ff_padded / DL_PIECE;
-  auto addr = [&](int pair, int piece, int r) -> const uint16_t* {
+  auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
     const int i = piece / per_expert, col = (piece - i * per_expert) * DL_PIECE + lane8;
-    if (col >= p.ff) return nullptr;
-    return p.down + (static_cast<int64_t>(ch.expert[i]) * p.k + 2 * pair + r) * p.ff + col;
+    ok0 = ok1 = col < p.ff;
+    p0 = p.down + (static_cast<int64_t>(ch.expert[i]) * p.k + 2 * pair) * p.ff + (ok0 ? col : 0);
+    p1 = p0 + p.ff;
   };
   const int pieces = ch.n * per_expert;
   const int ks_here = pieces < ks ? 1 : ks;
-  RowPairs<decltype(addr)> rp(addr, begin, pieces > 0 ? end : begin, pieces, ks_here);
-  uint4 b0[DL_UN][2], b1[DL_UN][2];
-  rp.load(b0);
-  rp.load(b1);
+  RowPairs<decltype(addr)> rp(addr, dd_smem, begin, pieces > 0 ? end : begin, pieces, ks_here);
+  rp.start();
   dependent_wait();
   dependent_trigger();
-  for (int i = 0; i < ch.n; ++i)
-    for (int c = threadIdx.x; c < ff_padded; c += DL_THREADS)
-      xs[i * ff_padded + c] = c < p.ff ? ch.weight[i] * p.act[static_cast<int64_t>(ch.slot[i]) * p.ff + c] : 0.f;
-  __syncthreads();
-  while (rp.more()) {
-    rp.consume(b0, xs, part, begin);
-    rp.load(b0);
-    rp.consume(b1, xs, part, begin);
-    rp.load(b1);
+  const int per4 = ff_padded / 4;
+  for (int v = threadIdx.x; v < ch.n * per4; v += DL_THREADS) {
+    const int i = v / per4, c = (v - i * per4) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < p.ff) a = *reinterpret_cast<const float4*>(p.act + static_cast<int64_t>(ch.slot[i]) * p.ff + c);
+    const float w = ch.weight[i];
+    *reinterpret_cast<float4*>(xs + i * ff_padded + staged_at(c)) = make_float4(w * a.x, w * a.y, w * a.z, w * a.w);
   }
+  __syncthreads();
+  rp.run(xs, part);
   __syncthreads();
   for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS) {
     const int row = begin * 2 + i;
@@ -695,9 +802,8 @@ int decode_experts(const DecodeExperts& a, cudaStream_t st) {
     const int pieces = (a.k + DL_PIECE - 1) / DL_PIECE, padded = pieces * DL_PIECE, pairs = a.r.top * a.ff;
     const int grid = pairs < sm_count() ? pairs : sm_count();
     const int per = (pairs + grid - 1) / grid, ks = pick_ks(per, pieces);
-    const int smem = (padded + per * 2 * ks) * static_cast<int>(sizeof(float));
-    if (smem > 48 * 1024 && (s = ensure_dynamic_smem(reinterpret_cast<const void*>(decode_gate_up_kernel), smem)) != YTC_OK)
-      return s;
+    const int smem = DL_WARPS * DL_RING + (padded + per * 2 * ks) * static_cast<int>(sizeof(float));
+    if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_gate_up_kernel), smem, "an expert's input")) != YTC_OK) return s;
     YTC_CUDA(launch_overlapped(decode_gate_up_kernel, dim3(grid), dim3(DL_THREADS), smem, st, a, ks, padded));
     count_launch();
     YTC_CUDA(cudaGetLastError());
@@ -705,13 +811,8 @@ int decode_experts(const DecodeExperts& a, cudaStream_t st) {
   const int per_expert = (a.ff + DL_PIECE - 1) / DL_PIECE, ff_padded = per_expert * DL_PIECE, pairs = a.k / 2;
   const int grid = pairs < sm_count() ? pairs : sm_count();
   const int per = (pairs + grid - 1) / grid, ks = pick_ks(per, a.r.top * per_expert);
-  const int smem = (a.r.top * ff_padded + per * 2 * ks) * static_cast<int>(sizeof(float));
-  if (smem > 220 * 1024) {
-    set_last_error("decode step: %d experts of %d channels do not fit shared memory", a.r.top, a.ff);
-    return YTC_UNSUPPORTED;
-  }
-  if (smem > 48 * 1024 && (s = ensure_dynamic_smem(reinterpret_cast<const void*>(decode_down_kernel), smem)) != YTC_OK)
-    return s;
+  const int smem = DL_WARPS * DL_RING + (a.r.top * ff_padded + per * 2 * ks) * static_cast<int>(sizeof(float));
+  if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_down_kernel), smem, "the experts' activations")) != YTC_OK) return s;
   YTC_CUDA(launch_overlapped(decode_down_kernel, dim3(grid), dim3(DL_THREADS), smem, st, a, ks, ff_padded));
   count_launch();
   YTC_CUDA(cudaGetLastError());

@@ -159,89 +159,107 @@ inline int moe_max_tiles(int64_t rows, const RouterSpec& r) {
 }
 
 #ifdef __CUDACC__
+// Floats as unsigned integers in the same order; minus infinity is above 0.
+__device__ __forceinline__ uint32_t ordered_key(float f) {
+  const uint32_t u = __float_as_uint(f);
+  return (u & 0x80000000u) ? ~u : (u | 0x80000000u);
+}
+// One warp takes the largest of its keys (VPL per lane, number j * 32 + lane; equal keys: the lowest number) and
+// removes it. False when only keys up to `floor` are left.
+template <int VPL>
+__device__ __forceinline__ bool warp_take_largest(uint32_t (&key)[VPL], int lane, uint32_t floor, int& index) {
+  uint32_t best = 0;
+  int bj = 0;
+#pragma unroll
+  for (int j = 0; j < VPL; ++j)
+    if (key[j] > best) {
+      best = key[j];
+      bj = j;
+    }
+  const uint32_t top = __reduce_max_sync(0xffffffffu, best);
+  if (top <= floor) return false;
+  index = static_cast<int>(__reduce_min_sync(0xffffffffu, best == top ? static_cast<uint32_t>(bj * 32 + lane) : 0xffffffffu));
+#pragma unroll
+  for (int j = 0; j < VPL; ++j)
+    if (j * 32 + lane == index) key[j] = 0;
+  return true;
+}
+
 // One warp routes one token. s: logits of the token in shared memory (overwritten by the scores), c: as many floats of
-// scratch. Afterwards lane k < top holds the k-th choice (-1: none) and its weight.
+// scratch; at most 32 * VPL routes. Afterwards lane k < top holds the k-th choice (-1: none) and its weight.
+template <int VPL>
 __device__ __forceinline__ void warp_route(float* s, float* c, const float* correction, const RouterSpec& r, int lane,
                                            int& choice, float& weight) {
   const int n = r.experts + r.identity;
+  const uint32_t floor = ordered_key(-INFINITY);
+  float v[VPL];
   float m = -INFINITY;
-  for (int i = lane; i < n; i += 32) m = fmaxf(m, s[i]);
+#pragma unroll
+  for (int j = 0; j < VPL; ++j) {
+    const int i = j * 32 + lane;
+    v[j] = i < n ? s[i] : -INFINITY;
+    m = fmaxf(m, v[j]);
+  }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
   float sum = 0.f;
-  for (int i = lane; i < n; i += 32) {
-    const float e = expf(s[i] - m);
-    s[i] = e;
-    sum += e;
+#pragma unroll
+  for (int j = 0; j < VPL; ++j) {
+    v[j] = j * 32 + lane < n ? expf(v[j] - m) : 0.f;
+    sum += v[j];
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-  for (int i = lane; i < n; i += 32) {
-    const float p = s[i] / sum;
-    s[i] = p;
-    c[i] = p + correction[i];
+  uint32_t key[VPL];
+#pragma unroll
+  for (int j = 0; j < VPL; ++j) {
+    const int i = j * 32 + lane;
+    key[j] = 0;
+    if (i < n) {
+      const float p = v[j] / sum, choice_score = p + correction[i];
+      s[i] = p;
+      c[i] = choice_score;
+      key[j] = ordered_key(choice_score);
+    }
   }
   __syncwarp();
   if (r.keep < r.count) {
-    // a group is kept when fewer than `keep` groups are better (larger score, then smaller index)
     const int per = n / r.count;
-    float g_best[LM_MAX_ROUTES / 32];  // (registers: groups lane, lane + 32, ...)
-    const int rounds = (r.count + 31) / 32;
-#pragma unroll 1
-    for (int q = 0; q < rounds; ++q) {
-      const int g = q * 32 + lane;
+    uint32_t gkey[VPL];
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+      const int g = j * 32 + lane;
       float b = -INFINITY;
       if (g < r.count)
         for (int i = 0; i < per; ++i) b = fmaxf(b, c[g * per + i]);
-      g_best[q] = b;
-    }
-    uint32_t dead[LM_MAX_ROUTES / 32];
-#pragma unroll 1
-    for (int q = 0; q < rounds; ++q) {
-      const int g = q * 32 + lane;
-      int better = 0;
-      for (int q2 = 0; q2 < rounds; ++q2)
-        for (int l = 0; l < 32; ++l) {
-          const int g2 = q2 * 32 + l;
-          if (g2 >= r.count) break;
-          const float b2 = __shfl_sync(0xffffffffu, g_best[q2], l);
-          better += (b2 > g_best[q] || (b2 == g_best[q] && g2 < g)) ? 1 : 0;
-        }
-      dead[q] = __ballot_sync(0xffffffffu, g < r.count && better >= r.keep);
+      gkey[j] = g < r.count ? ordered_key(b) : 0;
     }
     __syncwarp();
-    for (int i = lane; i < n; i += 32) {
-      const int g = i / per;
-      if (g < r.count && ((dead[g >> 5] >> (g & 31)) & 1u)) c[i] = -INFINITY;
+#pragma unroll
+    for (int j = 0; j < VPL; ++j)
+      if (j * 32 + lane < r.count) c[j * 32 + lane] = 0.f;  // from here on: 1 marks a kept group
+    __syncwarp();
+    for (int k = 0; k < r.keep; ++k) {
+      int g = 0;
+      if (!warp_take_largest<VPL>(gkey, lane, 0, g)) break;
+      if (lane == 0) c[g] = 1.f;
     }
     __syncwarp();
+#pragma unroll
+    for (int j = 0; j < VPL; ++j) {
+      const int i = j * 32 + lane;
+      if (i < n && c[i / per] == 0.f) key[j] = floor;
+    }
   }
   choice = -1;
   weight = 0.f;
   for (int k = 0; k < r.top; ++k) {
-    float b = -INFINITY;
-    int bi = 0x7fffffff;
-    for (int i = lane; i < n; i += 32)
-      if (c[i] > b) {  // (ascending i: the first of equals is kept)
-        b = c[i];
-        bi = i;
-      }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ob = __shfl_xor_sync(0xffffffffu, b, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-      if (ob > b || (ob == b && oi < bi)) {
-        b = ob;
-        bi = oi;
-      }
-    }
-    const bool found = bi < n;  // (nothing left to choose: every remaining choice score is minus infinity)
+    int i = 0;
+    if (!warp_take_largest<VPL>(key, lane, floor, i)) break;
     if (lane == k) {
-      choice = found ? bi : -1;
-      weight = found ? s[bi] : 0.f;
+      choice = i;
+      weight = s[i];
     }
-    if (found && lane == (bi & 31)) c[bi] = -INFINITY;
-    __syncwarp();
   }
 }
 #endif

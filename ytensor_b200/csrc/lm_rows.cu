@@ -160,38 +160,38 @@ int residual_norm(const ResidualNorm& a, cudaStream_t st) {
 }
 
 // ------------------------------------------------------------------ K/V append
-// One 8-element piece of a key or value vector per thread.
+// One row (token) per CTA at a time, one 8-element piece of a key or value vector per thread.
+constexpr int AK_THREADS = 128;
 template <typename T>
-__global__ void __launch_bounds__(256) append_kv_kernel(const AppendKv p) {
+__global__ void __launch_bounds__(AK_THREADS) append_kv_kernel(const AppendKv p) {
   dependent_wait();
   dependent_trigger();
-  const int kp = p.kv_heads * p.dim / 8, vp = p.kv_heads * p.vdim / 8, per_row = kp + vp;
-  const int64_t total = static_cast<int64_t>(p.batch) * p.len * per_row;
+  const int kp = p.kv_heads * p.dim / 8, vp = p.kv_heads * p.vdim / 8;
+  const int rows = p.batch * p.len;
   const float lam = p.mix == VMIX_MIX ? *p.lambda : 0.f;
-  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
-       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
-    const int64_t row = i / per_row;
-    const int c = static_cast<int>(i - row * per_row);
-    const int b = static_cast<int>(row / p.len), t = static_cast<int>(row - static_cast<int64_t>(b) * p.len);
+  for (int row = blockIdx.x; row < rows; row += gridDim.x) {
+    const int b = row / p.len, t = row - b * p.len;
     const int64_t ring_row = (p.pos0 + t) % p.ring;
     const T* src = static_cast<const T*>(p.qkv) + row * p.ld;
-    float f[8];
-    if (c < kp) {
-      const int e = c * 8, g = e / p.dim, d = e - g * p.dim;
-      Vec8<T>::load(src + p.k_off + e, f);
-      Vec8<T>::store(static_cast<T*>(p.k) + ((static_cast<int64_t>(b) * p.kv_heads + g) * p.ring + ring_row) * p.dim + d, f);
-    } else {
-      const int e = (c - kp) * 8, g = e / p.vdim, d = e - g * p.vdim;
-      Vec8<T>::load(src + p.v_off + e, f);
-      T* first = static_cast<T*>(p.v_first) + row * (static_cast<int64_t>(p.kv_heads) * p.vdim) + e;
-      if (p.mix == VMIX_FIRST) Vec8<T>::store(first, f);
-      if (p.mix == VMIX_MIX) {
-        float v0[8];
-        Vec8<T>::load(first, v0);
+    for (int c = threadIdx.x; c < kp + vp; c += AK_THREADS) {
+      float f[8];
+      if (c < kp) {
+        const int e = c * 8, g = e / p.dim, d = e - g * p.dim;
+        Vec8<T>::load(src + p.k_off + e, f);
+        Vec8<T>::store(static_cast<T*>(p.k) + ((static_cast<int64_t>(b) * p.kv_heads + g) * p.ring + ring_row) * p.dim + d, f);
+      } else {
+        const int e = (c - kp) * 8, g = e / p.vdim, d = e - g * p.vdim;
+        Vec8<T>::load(src + p.v_off + e, f);
+        T* first = static_cast<T*>(p.v_first) + row * (static_cast<int64_t>(p.kv_heads) * p.vdim) + e;
+        if (p.mix == VMIX_FIRST) Vec8<T>::store(first, f);
+        if (p.mix == VMIX_MIX) {
+          float v0[8];
+          Vec8<T>::load(first, v0);
 #pragma unroll
-        for (int k = 0; k < 8; ++k) f[k] = (1.f - lam) * f[k] + lam * v0[k];
+          for (int k = 0; k < 8; ++k) f[k] = (1.f - lam) * f[k] + lam * v0[k];
+        }
+        Vec8<T>::store(static_cast<T*>(p.v) + ((static_cast<int64_t>(b) * p.kv_heads + g) * p.ring + ring_row) * p.vdim + d, f);
       }
-      Vec8<T>::store(static_cast<T*>(p.v) + ((static_cast<int64_t>(b) * p.kv_heads + g) * p.ring + ring_row) * p.vdim + d, f);
     }
   }
 }
@@ -200,10 +200,9 @@ int append_kv(const AppendKv& a, cudaStream_t st) {
   YTC_REQUIRE(a.dim % 8 == 0 && a.vdim % 8 == 0 && a.ld % 8 == 0 && a.k_off % 8 == 0 && a.v_off % 8 == 0 && a.len <= a.ring,
               "append_kv: bad extent");
   YTC_REQUIRE(a.mix == VMIX_NONE || a.v_first, "append_kv: no place for the first layer's values");
-  const int64_t total = static_cast<int64_t>(a.batch) * a.len * a.kv_heads * (a.dim + a.vdim) / 8;
-  const int64_t blocks = (total + 255) / 256, cap = static_cast<int64_t>(sm_count()) * 16;
+  const int64_t blocks = static_cast<int64_t>(a.batch) * a.len, cap = static_cast<int64_t>(sm_count()) * 16;
   YTC_CUDA(launch_overlapped(a.dtype == YTC_BF16 ? append_kv_kernel<uint16_t> : append_kv_kernel<float>,
-                             dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)), dim3(256), 0, st, a));
+                             dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)), dim3(AK_THREADS), 0, st, a));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;

@@ -8,6 +8,7 @@ namespace ytk {
 
 constexpr int MR_WARPS = 4;
 
+template <int VPL>
 __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const float* logits, int64_t ld, const float* correction,
                                                                   int64_t rows, const RouterSpec r, int* choice,
                                                                   float* weight, int* rank, int* count) {
@@ -23,7 +24,7 @@ __global__ void __launch_bounds__(MR_WARPS * 32) moe_route_kernel(const float* l
     __syncwarp();
     int c;
     float w;
-    warp_route(s, s + n, correction, r, lane, c, w);
+    warp_route<VPL>(s, s + n, correction, r, lane, c, w);
     if (lane < r.top) {
       choice[row * r.top + lane] = c;
       weight[row * r.top + lane] = w;
@@ -41,7 +42,8 @@ int moe_route(const float* logits, int64_t ld, const float* correction, int64_t 
               r.identity, r.top, r.keep, r.count, LM_MAX_ROUTES, LM_MAX_TOP);
   if (rows <= 0) return YTC_OK;
   const int64_t blocks = (rows + MR_WARPS - 1) / MR_WARPS, cap = static_cast<int64_t>(sm_count()) * 8;
-  YTC_CUDA(launch_overlapped(moe_route_kernel, dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)),
+  auto* fn = n <= 128 ? moe_route_kernel<4> : n <= 256 ? moe_route_kernel<8> : moe_route_kernel<LM_MAX_ROUTES / 32>;
+  YTC_CUDA(launch_overlapped(fn, dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)),
                              dim3(MR_WARPS * 32), MR_WARPS * 2 * n * sizeof(float), st, logits, ld, correction, rows, r,
                              choice, weight, rank, count));
   count_launch();
