@@ -14,9 +14,9 @@
 
 namespace ytk {
 
-constexpr int DL_THREADS = 256, DL_WARPS = DL_THREADS / 32;
+constexpr int DL_THREADS = 512, DL_WARPS = DL_THREADS / 32;
 constexpr int DL_PIECE = 256;              // columns a warp covers with one 16-byte load per lane
-constexpr int DL_DEPTH = 8;                // row-pair pieces in flight per warp
+constexpr int DL_DEPTH = 4;                // row-pair pieces in flight per warp
 constexpr int DL_RING = DL_DEPTH * 2 * 512;  // bytes of a warp's weight ring
 
 // ---------------------------------------------------------------- asynchronous copies of 16 bytes per lane
@@ -221,7 +221,7 @@ static int pick_ks(int pairs_per_cta, int pieces) {
   for (int ks = 1; ks <= DL_WARPS && ks <= pieces; ks *= 2) {
     const int slots = DL_WARPS / ks;
     const double rounds = (pairs_per_cta + slots - 1) / slots;
-    const double cost = rounds * ((pieces + ks - 1) / ks);
+    const double cost = rounds * ((pieces + ks - 1) / ks + 2);  // (the sum over the lanes costs about two pieces)
     if (cost < best_cost * 0.95) {
       best_cost = cost;
       best = ks;
@@ -248,7 +248,7 @@ static int check_input(const DecodeInput& in, int k) {
 }
 
 // ------------------------------------------------------------------ linear
-__global__ void __launch_bounds__(DL_THREADS) decode_linear_kernel(const DecodeLinear p, int ks, int padded) {
+__global__ void __launch_bounds__(DL_THREADS, 2) decode_linear_kernel(const DecodeLinear p, int ks, int padded) {
   extern __shared__ __align__(16) uint8_t dl_smem[];  // weight rings, input, part[]
   __shared__ float red[2 * DL_WARPS];
   const InputSmem in = input_smem(reinterpret_cast<float*>(dl_smem + DL_WARPS * DL_RING), p.k, padded);
@@ -296,23 +296,15 @@ int decode_linear(const DecodeLinear& a, cudaStream_t st) {
 }
 
 // ------------------------------------------------------------------ attention
-// One cluster of CTAs per K/V head and block of up to four query heads of its group; the keys of the window are split
-// over all warps of the cluster. A warp works on its own: it copies DA_KW keys and values at a time into its part of
+// One cluster of CTAs per K/V head and block of one, two or four query heads of its group; the keys of the window are
+// split over all warps of the cluster. A warp works on its own: it copies DA_KW keys and values at a time into its part of
 // shared memory (the first ones requested before the wait for the projection), takes the scores with eight lanes per
-// key, and sums the values with the value dim across its lanes. Warps meet through shared memory, CTAs through
-// distributed shared memory.
+// key, and sums the values with the value dim across its lanes. Warps meet through shared memory; the CTAs push their
+// results into the shared memory of the cluster's first CTA, which adds them.
 constexpr int DA_MAX_CLUSTER = 8;
-constexpr int DA_GB = 4;  // query heads per cluster
 template <typename T>
-constexpr int DA_KW = sizeof(T) == 2 ? 16 : 8;  // keys per step of a warp
+constexpr int DA_KW = sizeof(T) == 2 ? 8 : 4;  // keys per step of a warp
 
-__device__ __forceinline__ float ld_cluster(const float* p, uint32_t rank) {
-  uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(p)), r;
-  float v;
-  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(rank));
-  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(r) : "memory");
-  return v;
-}
 __device__ __forceinline__ void cluster_barrier() {
   asm volatile("barrier.cluster.arrive.release.aligned;" ::: "memory");
   asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
@@ -329,22 +321,33 @@ __device__ __forceinline__ void load4(const T* p, float (&f)[4]) {
   }
 }
 
-// NV: float4 slots of the value dim per lane (1: up to 128, 2: up to 256).
-template <typename T, int NV>
-__global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAttn p, int ncta, int nbuf) {
-  constexpr int KW = DA_KW<T>, GB = DA_GB;
-  // K/V of the warps [warps][nbuf][KW][dim + vdim] (T), q[GB][dim], o[warps][GB][vdim] (merged into o[0])
+// Stores to the shared memory of CTA `rank` of the cluster.
+__device__ __forceinline__ void st_cluster(float* p, uint32_t rank, float v) {
+  uint32_t a = static_cast<uint32_t>(__cvta_generic_to_shared(p)), r;
+  asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(r) : "r"(a), "r"(rank));
+  asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(r), "f"(v) : "memory");
+}
+
+// NH: query heads per cluster, NV: float4 slots of the value dim per lane (1: up to 128, 2: up to 256).
+template <typename T, int NH, int NV>
+__global__ void __launch_bounds__(DL_THREADS, NV == 1 ? 2 : 1) decode_attn_kernel(const DecodeAttn p, int ncta, int nbuf) {
+  constexpr int KW = DA_KW<T>;
+  // K/V of the warps [warps][nbuf][KW][dim + vdim] (T), q[NH][dim], o[warps][NH][vdim], the CTAs' results
+  // x[cluster][NH][vdim] (in CTA 0)
   extern __shared__ __align__(16) uint8_t da_smem[];
-  __shared__ float w_s[DL_WARPS][GB][KW], al_s[DL_WARPS][GB], m_s[DL_WARPS][GB], l_s[DL_WARPS][GB], cm[GB], cl[GB];
+  __shared__ float w_s[DL_WARPS][NH][KW], al_s[DL_WARPS][NH], m_s[DL_WARPS][NH], l_s[DL_WARPS][NH];
+  __shared__ float xm[DA_MAX_CLUSTER][NH], xl[DA_MAX_CLUSTER][NH];
   const int D = p.dim, Dv = p.vdim, row_e = D + Dv;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   T* kv_s = reinterpret_cast<T*>(da_smem) + static_cast<size_t>(warp) * nbuf * KW * row_e;
   float* q_s = reinterpret_cast<float*>(da_smem + static_cast<size_t>(DL_WARPS) * nbuf * KW * row_e * sizeof(T));
-  float* o_s = q_s + GB * D;
+  float* o_s = q_s + NH * D;
+  float* x_s = o_s + (DL_WARPS * NH * Dv > row_e ? DL_WARPS * NH * Dv : row_e);
   const int unit = blockIdx.x / ncta, rank = blockIdx.x - unit * ncta;
-  const int blocks = (p.groups + GB - 1) / GB;
-  const int g = unit / blocks, h0 = (unit - g * blocks) * GB;  // K/V head, first query head of the group
-  const int nh = p.groups - h0 < GB ? p.groups - h0 : GB;
+  const int blocks = (p.groups + NH - 1) / NH;
+  const int g = unit / blocks, h0 = (unit - g * blocks) * NH;  // K/V head, first query head of the group
+  const int nh = p.groups - h0 < NH ? p.groups - h0 : NH;
+  if (ncta > 1) asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // (this CTA has started)
 
   // (the position word was written before this step's first kernel started)
   const int pos = *p.pos;
@@ -375,6 +378,7 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
   };
   fetch(0, 0);
   if (nbuf > 1) fetch(KW, 1);
+  const float lam = p.mix == VMIX_MIX ? *p.lambda : 0.f;
   dependent_wait();
   dependent_trigger();
   const int H = p.kv_heads * p.groups;
@@ -384,7 +388,6 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
   if (has_new) {  // the new key and value: behind the warp's old keys, and (one cluster per K/V head) into the rings
     const float* k_new = p.qkv + static_cast<int64_t>(H) * D + static_cast<int64_t>(g) * D;
     const float* v_new = p.qkv + static_cast<int64_t>(H + p.kv_heads) * D + static_cast<int64_t>(g) * Dv;
-    const float lam = p.mix == VMIX_MIX ? *p.lambda : 0.f;
     const int64_t row = pos % p.ring;
     T* kw = static_cast<T*>(p.k) + (static_cast<int64_t>(g) * p.ring + row) * D;
     T* vw = static_cast<T*>(p.v) + (static_cast<int64_t>(g) * p.ring + row) * Dv;
@@ -395,8 +398,8 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
       if (e < D) {
         Vec8<float>::load(k_new + e, f);
       } else {
-        Vec8<float>::load(v_new + e - D, f);
         float* first = p.v_first + static_cast<int64_t>(g) * Dv + e - D;
+        Vec8<float>::load(v_new + e - D, f);
         if (p.mix == VMIX_FIRST && first_block) Vec8<float>::store(first, f);
         if (p.mix == VMIX_MIX) {
           float v0[8];
@@ -409,13 +412,12 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
       Vec8<float>::store(o_s + e, f);  // joins the keys in shared memory when their last step is reached
     }
   }
-  __syncthreads();
-  float acc[GB][NV * 4] = {};
-  if (lane < GB) {
+  if (lane < NH) {
     m_s[warp][lane] = -CUDART_INF_F;
     l_s[warp][lane] = 0.f;
   }
-  __syncwarp();
+  __syncthreads();
+  float acc[NH][NV * 4] = {};
 #pragma unroll 1
   for (int c0 = 0, buf = 0; c0 < mine; c0 += KW, buf = (buf + 1 == nbuf ? 0 : buf + 1)) {
     const int n = mine - c0 < KW ? mine - c0 : KW;
@@ -435,12 +437,12 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
     for (int key0 = 0; key0 < n; key0 += 4) {
       const int key = key0 + (lane >> 3);
       const T* k = kv + (key < n ? key : 0) * row_e;
-      float dot[GB] = {};
+      float dot[NH] = {};
       for (int c = (lane & 7) * 8; c < D; c += 64) {
         float a[8];
         Vec8<T>::load(k + c, a);
 #pragma unroll
-        for (int h = 0; h < GB; ++h) {
+        for (int h = 0; h < NH; ++h) {
           if (h >= nh) break;
           float b[8];
           Vec8<float>::load(q_s + h * D + c, b);
@@ -449,8 +451,7 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
         }
       }
 #pragma unroll
-      for (int h = 0; h < GB; ++h) {
-        if (h >= nh) break;
+      for (int h = 0; h < NH; ++h) {
         dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 1);
         dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 2);
         dot[h] += __shfl_xor_sync(0xffffffffu, dot[h], 4);
@@ -460,8 +461,9 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
     __syncwarp();
     // weights: KW lanes per head
 #pragma unroll 1
-    for (int h = lane / KW; h < GB; h += 32 / KW) {
-      const int key = lane % KW;
+    for (int hb = 0; hb < nh; hb += 32 / KW) {
+      const int h = hb + lane / KW, key = lane % KW;
+      const int hc = h < nh ? h : 0;
       float s = -CUDART_INF_F;
       if (h < nh && key < n) {
         s = w_s[warp][h][key];
@@ -470,23 +472,26 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
       float m = s;
 #pragma unroll
       for (int o = KW / 2; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-      const float m_old = m_s[warp][h], m_new = fmaxf(m_old, m);
+      const float m_old = m_s[warp][hc], m_new = fmaxf(m_old, m);
       const float w = s == -CUDART_INF_F ? 0.f : expf(s - m_new);
       float l = w;
 #pragma unroll
       for (int o = KW / 2; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-      w_s[warp][h][key] = w;
-      if (key == 0) {
-        const float alpha = m_old == -CUDART_INF_F ? 0.f : expf(m_old - m_new);
-        al_s[warp][h] = alpha;
-        m_s[warp][h] = m_new;
-        l_s[warp][h] = l_s[warp][h] * alpha + l;
+      __syncwarp();
+      if (h < nh) {
+        w_s[warp][h][key] = w;
+        if (key == 0) {
+          const float alpha = m_old == -CUDART_INF_F ? 0.f : expf(m_old - m_new);
+          al_s[warp][h] = alpha;
+          m_s[warp][h] = m_new;
+          l_s[warp][h] = l_s[warp][h] * alpha + l;
+        }
       }
     }
     __syncwarp();
 #pragma unroll
-    for (int h = 0; h < GB; ++h) {
-      const float alpha = al_s[warp][h];
+    for (int h = 0; h < NH; ++h) {
+      const float alpha = h < nh ? al_s[warp][h] : 0.f;
 #pragma unroll
       for (int e = 0; e < NV * 4; ++e) acc[h][e] *= alpha;
     }
@@ -497,8 +502,8 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
       for (int j = 0; j < NV; ++j)
         if (j * 128 + lane * 4 < Dv) load4<T>(kv + key * row_e + D + j * 128 + lane * 4, v[j]);
 #pragma unroll
-      for (int h = 0; h < GB; ++h) {
-        const float w = w_s[warp][h][key];
+      for (int h = 0; h < NH; ++h) {
+        const float w = h < nh ? w_s[warp][h][key] : 0.f;
 #pragma unroll
         for (int e = 0; e < NV * 4; ++e) acc[h][e] = fmaf(w, v[e >> 2][e & 3], acc[h][e]);
       }
@@ -508,62 +513,67 @@ __global__ void __launch_bounds__(DL_THREADS) decode_attn_kernel(const DecodeAtt
     else cp_async_commit();
   }
   __syncthreads();  // (the new key's copy in o_s has been read)
+  // The CTA's result: the warps' sums, brought to the CTA's maximum by every warp itself.
+  float mc[NH];
 #pragma unroll
-  for (int h = 0; h < GB; ++h)
+  for (int h = 0; h < NH; ++h) {
+    float m = lane < DL_WARPS ? m_s[lane][h] : -CUDART_INF_F;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+    mc[h] = m;
+    const float f = m_s[warp][h] == -CUDART_INF_F ? 0.f : expf(m_s[warp][h] - m);
 #pragma unroll
     for (int j = 0; j < NV; ++j)
       if (j * 128 + lane * 4 < Dv)
-        *reinterpret_cast<float4*>(o_s + (warp * GB + h) * Dv + j * 128 + lane * 4) =
-            make_float4(acc[h][4 * j], acc[h][4 * j + 1], acc[h][4 * j + 2], acc[h][4 * j + 3]);
+        *reinterpret_cast<float4*>(o_s + (warp * NH + h) * Dv + j * 128 + lane * 4) =
+            make_float4(f * acc[h][4 * j], f * acc[h][4 * j + 1], f * acc[h][4 * j + 2], f * acc[h][4 * j + 3]);
+  }
   __syncthreads();
-  // the CTA's result, then the cluster's: each CTA finishes a share of the outputs
+  // ... goes to CTA 0 of the cluster, which adds the CTAs'
+  if (ncta > 1) asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
   for (int i = threadIdx.x; i < nh * Dv; i += DL_THREADS) {
-    const int h = i / Dv;
+    float o = 0.f;
+#pragma unroll
+    for (int w = 0; w < DL_WARPS; ++w) o += o_s[w * NH * Dv + i];
+    if (ncta > 1) st_cluster(x_s + rank * NH * Dv + i, 0, o);
+    else x_s[i] = o;
+  }
+  if (warp < nh) {
+    const int h = warp;
+    const float ml = lane < DL_WARPS ? m_s[lane][h] : -CUDART_INF_F;
     float m = -CUDART_INF_F;
 #pragma unroll
-    for (int w = 0; w < DL_WARPS; ++w) m = fmaxf(m, m_s[w][h]);
-    float l = 0.f, o = 0.f;
+    for (int k = 0; k < NH; ++k) m = k == h ? mc[k] : m;
+    float l = ml == -CUDART_INF_F ? 0.f : expf(ml - m) * l_s[lane][h];
 #pragma unroll
-    for (int w = 0; w < DL_WARPS; ++w) {
-      const float f = m_s[w][h] == -CUDART_INF_F ? 0.f : expf(m_s[w][h] - m);
-      l = fmaf(f, l_s[w][h], l);
-      o = fmaf(f, o_s[w * GB * Dv + i], o);
-    }
-    o_s[i] = o;  // (the element of warp 0 that this thread alone has read)
-    if (i == h * Dv) {
-      cm[h] = m;
-      cl[h] = l;
+    for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+    if (lane == 0) {
+      if (ncta > 1) {
+        st_cluster(&xm[rank][h], 0, m);
+        st_cluster(&xl[rank][h], 0, l);
+      } else {
+        xm[0][h] = m;
+        xl[0][h] = l;
+      }
     }
   }
   if (ncta > 1) cluster_barrier();
   else __syncthreads();
+  if (rank != 0) return;
   float* out = p.out + static_cast<int64_t>(g * p.groups + h0) * Dv;
-  for (int i = rank * DL_THREADS + threadIdx.x; i < nh * Dv; i += ncta * DL_THREADS) {
+  for (int i = threadIdx.x; i < nh * Dv; i += DL_THREADS) {
     const int h = i / Dv;
-    if (ncta == 1) {
-      out[i] = o_s[i] / cl[h];
-      continue;
-    }
-    float ms[DA_MAX_CLUSTER], ls[DA_MAX_CLUSTER], os[DA_MAX_CLUSTER], m = -CUDART_INF_F;
-#pragma unroll
-    for (int r = 0; r < DA_MAX_CLUSTER; ++r) {
-      const uint32_t from = r < ncta ? r : 0;
-      ms[r] = ld_cluster(cm + h, from);
-      ls[r] = ld_cluster(cl + h, from);
-      os[r] = ld_cluster(o_s + i, from);
-      if (r >= ncta) ms[r] = -CUDART_INF_F;
-      m = fmaxf(m, ms[r]);
-    }
+    float m = -CUDART_INF_F;
+    for (int r = 0; r < ncta; ++r) m = fmaxf(m, xm[r][h]);
     float l = 0.f, o = 0.f;
-#pragma unroll
-    for (int r = 0; r < DA_MAX_CLUSTER; ++r) {
-      const float f = ms[r] == -CUDART_INF_F ? 0.f : expf(ms[r] - m);
-      l = fmaf(f, ls[r], l);
-      o = fmaf(f, os[r], o);
+#pragma unroll 4
+    for (int r = 0; r < ncta; ++r) {
+      const float f = xm[r][h] == -CUDART_INF_F ? 0.f : expf(xm[r][h] - m);
+      l = fmaf(f, xl[r][h], l);
+      o = fmaf(f, x_s[r * NH * Dv + i], o);
     }
     out[i] = o / l;
   }
-  if (ncta > 1) cluster_barrier();  // no CTA leaves while another may still read its shared memory
 }
 
 // Launch with an optional cluster size, dependent on the kernel before it inside an overlap scope.
@@ -586,21 +596,21 @@ static cudaError_t launch_cluster(void (*kernel)(KArgs...), int grid, int cluste
   return cudaLaunchKernelEx(&cfg, kernel, static_cast<KArgs>(args)...);
 }
 
-template <typename T>
+template <typename T, int NH>
 static int decode_attention_t(const DecodeAttn& a, cudaStream_t st) {
   constexpr int KW = DA_KW<T>;
-  const int units = a.kv_heads * ((a.groups + DA_GB - 1) / DA_GB);
+  const int units = a.kv_heads * ((a.groups + NH - 1) / NH);
   int ncta = 1;
   while (ncta < DA_MAX_CLUSTER && static_cast<int64_t>(ncta) * DL_WARPS * 4 < a.max_keys && units * ncta * 2 <= sm_count())
     ncta *= 2;
-  const int64_t per_warp = (a.max_keys + ncta * DL_WARPS - 1) / (ncta * DL_WARPS) + 1;
+  const int64_t per_warp = (a.max_keys - 1) / (ncta * DL_WARPS) + 1;
   const int step = DL_WARPS * KW * (a.dim + a.vdim) * static_cast<int>(sizeof(T));
-  // (the new key and value pass through the output area on their way)
-  const int outs = DL_WARPS * DA_GB * a.vdim > a.dim + a.vdim ? DL_WARPS * DA_GB * a.vdim : a.dim + a.vdim;
-  const int rest = (DA_GB * a.dim + outs) * 4;
-  const int nbuf = (per_warp > KW && 2 * step + rest <= 150 * 1024) ? 2 : 1;
+  // (the new key and value pass through the warps' output area on their way)
+  const int outs = DL_WARPS * NH * a.vdim > a.dim + a.vdim ? DL_WARPS * NH * a.vdim : a.dim + a.vdim;
+  const int rest = (NH * a.dim + outs + ncta * NH * a.vdim) * 4;
+  const int nbuf = (per_warp > KW && 2 * step + rest <= 170 * 1024) ? 2 : 1;
   const int smem = nbuf * step + rest;
-  auto* fn = a.vdim <= 128 ? decode_attn_kernel<T, 1> : decode_attn_kernel<T, 2>;
+  auto* fn = a.vdim <= 128 ? decode_attn_kernel<T, NH, 1> : decode_attn_kernel<T, NH, 2>;
   const int s = dl_smem_check(reinterpret_cast<const void*>(fn), smem, "attention");
   if (s != YTC_OK) return s;
   YTC_CUDA(launch_cluster(fn, units * ncta, ncta, smem, st, a, ncta, nbuf));
@@ -612,22 +622,92 @@ static int decode_attention_t(const DecodeAttn& a, cudaStream_t st) {
 int decode_attention(const DecodeAttn& a, cudaStream_t st) {
   YTC_REQUIRE(a.dim > 0 && a.dim % 8 == 0 && a.vdim > 0 && a.vdim % 8 == 0 && a.vdim <= 256 && a.max_keys > 0 && a.ring > 0,
               "decode step: head dims must be multiples of 8, the value dim at most 256");
-  return a.dtype == YTC_BF16 ? decode_attention_t<uint16_t>(a, st) : decode_attention_t<float>(a, st);
+  if (a.dtype == YTC_BF16)
+    return a.groups == 1 ? decode_attention_t<uint16_t, 1>(a, st)
+                         : a.groups == 2 ? decode_attention_t<uint16_t, 2>(a, st) : decode_attention_t<uint16_t, 4>(a, st);
+  return a.groups == 1 ? decode_attention_t<float, 1>(a, st)
+                       : a.groups == 2 ? decode_attention_t<float, 2>(a, st) : decode_attention_t<float, 4>(a, st);
 }
 
 // ------------------------------------------------------------------ router
 // One cluster: every CTA computes a share of the logits, CTA 0 collects them and routes.
 constexpr int DR_CLUSTER = 8;
-template <int VPL>
-__global__ void __launch_bounds__(DL_THREADS) decode_route_kernel(const DecodeRoute p, int ks, int padded) {
-  extern __shared__ __align__(16) uint8_t dr_smem[];  // weight rings, input, part[], scores[n], choice scores[n]
+
+// The rule of warp_route (lm_ops.cuh) by a whole CTA: every route counts the routes in front of it, so that there is no
+// chain of one selection after the other. s: logits, overwritten by the scores; c, g: scratch of n and `count` floats.
+__device__ __forceinline__ float block_max(float v, float* red) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float m = red[0];
+#pragma unroll
+  for (int i = 1; i < DL_WARPS; ++i) m = fmaxf(m, red[i]);
+  return m;
+}
+__device__ __forceinline__ bool comes_before(float a, int i, float b, int j) { return a > b || (a == b && i < j); }
+__device__ __forceinline__ void block_route(float* s, float* c, float* g, float* red, const float* correction,
+                                            const RouterSpec& r, int* choice, float* weight) {
+  const int n = r.experts + r.identity;
+  float m = -INFINITY;
+  for (int i = threadIdx.x; i < n; i += DL_THREADS) m = fmaxf(m, s[i]);
+  m = block_max(m, red);
+  float sum = 0.f;
+  for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+    const float e = expf(s[i] - m);
+    s[i] = e;
+    sum += e;
+  }
+  sum = dl_block_sum(sum, red + DL_WARPS);
+  for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+    const float p = s[i] / sum;
+    s[i] = p;
+    c[i] = p + correction[i];
+  }
+  if (threadIdx.x < r.top) {  // (places that no route takes)
+    choice[threadIdx.x] = -1;
+    weight[threadIdx.x] = 0.f;
+  }
+  __syncthreads();
+  if (r.keep < r.count) {
+    const int per = n / r.count;
+    for (int k = threadIdx.x; k < r.count; k += DL_THREADS) {
+      float b = -INFINITY;
+      for (int i = 0; i < per; ++i) b = fmaxf(b, c[k * per + i]);
+      g[k] = b;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+      const int mine = i / per;
+      int before = 0;
+      for (int k = 0; k < r.count; ++k) before += comes_before(g[k], k, g[mine], mine) ? 1 : 0;
+      if (before >= r.keep) c[i] = -INFINITY;
+    }
+    __syncthreads();
+  }
+  for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+    const float mine = c[i];
+    if (mine == -INFINITY) continue;
+    int before = 0;
+#pragma unroll 4
+    for (int k = 0; k < n; ++k) before += comes_before(c[k], k, mine, i) ? 1 : 0;
+    if (before < r.top) {
+      choice[before] = i;
+      weight[before] = s[i];
+    }
+  }
+}
+
+__global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const DecodeRoute p, int ks, int padded) {
+  extern __shared__ __align__(16) uint8_t dr_smem[];  // weight rings, input, part[], scores[n], choice scores[n], groups
   __shared__ float red[2 * DL_WARPS];
   const int n = p.r.experts + p.r.identity, pairs = (n + 1) / 2;
   const InputSmem in = input_smem(reinterpret_cast<float*>(dr_smem + DL_WARPS * DL_RING), p.k, padded);
   float* part = in.h + padded + 3 * p.k;
   float* s = part + ((pairs + DR_CLUSTER - 1) / DR_CLUSTER) * 2 * ks;
   float* c = s + n;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float* g = c + n;
+  const int lane = threadIdx.x & 31;
   const int rank = blockIdx.x;
   int begin, end;
   my_pairs(pairs, begin, end);
@@ -641,35 +721,20 @@ __global__ void __launch_bounds__(DL_THREADS) decode_route_kernel(const DecodeRo
   RowPairs<decltype(addr)> rp(addr, dr_smem, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
   prefetch_input(p.in, p.k, in);
   rp.start();
-  if (rank == 0)  // (brings the correction into the L1 / L2 ahead of its use)
-    for (int i = threadIdx.x; i < n; i += DL_THREADS) c[i] = p.correction[i];
+  float* corr = g + p.r.count;
+  if (rank == 0)
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) corr[i] = p.correction[i];
+  asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // (this CTA has started)
   dependent_wait();
   dependent_trigger();
   stage_input<DL_DEPTH - 1>(p.in, p.k, padded, in, red, rank == 0, p.h);
   rp.run(in.h, part);
   __syncthreads();
+  asm volatile("barrier.cluster.wait.acquire.aligned;" ::: "memory");
   for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS)
-    if (begin * 2 + i < n) s[begin * 2 + i] = sum_sub(part, i, ks);
+    if (begin * 2 + i < n) st_cluster(s + begin * 2 + i, 0, sum_sub(part, i, ks));
   cluster_barrier();
-  if (rank == 0) {
-    for (int e = threadIdx.x; e < n; e += DL_THREADS) {
-      const int pair = e / 2;
-      int owner = 0;
-      while (pair >= static_cast<int>(static_cast<int64_t>(pairs) * (owner + 1) / DR_CLUSTER)) ++owner;
-      if (owner != 0) s[e] = ld_cluster(s + e, owner);
-    }
-    __syncthreads();
-    if (warp == 0) {
-      int choice;
-      float weight;
-      warp_route<VPL>(s, c, p.correction, p.r, lane, choice, weight);
-      if (lane < p.r.top) {
-        p.choice[lane] = choice;
-        p.weight[lane] = weight;
-      }
-    }
-  }
-  cluster_barrier();
+  if (rank == 0) block_route(s, c, g, red, corr, p.r, p.choice, p.weight);
 }
 
 int decode_route(const DecodeRoute& a, cudaStream_t st) {
@@ -679,11 +744,10 @@ int decode_route(const DecodeRoute& a, cudaStream_t st) {
   const int pieces = (a.k + DL_PIECE - 1) / DL_PIECE, padded = pieces * DL_PIECE;
   const int ks = pick_ks(per, pieces);
   const int smem = DL_WARPS * DL_RING +
-                   (input_floats(a.in.kind, a.k, padded) + per * 2 * ks + 2 * n) * static_cast<int>(sizeof(float));
-  auto* fn = n <= 128 ? decode_route_kernel<4> : n <= 256 ? decode_route_kernel<8> : decode_route_kernel<LM_MAX_ROUTES / 32>;
+                   (input_floats(a.in.kind, a.k, padded) + per * 2 * ks + 3 * n + a.r.count) * static_cast<int>(sizeof(float));
   YTC_REQUIRE(a.in.kind != 2, "decode step: the router's input is a normed residual row");
-  if ((s = dl_smem_check(reinterpret_cast<const void*>(fn), smem, "the router")) != YTC_OK) return s;
-  YTC_CUDA(launch_cluster(fn, DR_CLUSTER, DR_CLUSTER, smem, st, a, ks, padded));
+  if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_route_kernel), smem, "the router")) != YTC_OK) return s;
+  YTC_CUDA(launch_cluster(decode_route_kernel, DR_CLUSTER, DR_CLUSTER, smem, st, a, ks, padded));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
@@ -722,7 +786,7 @@ __device__ __forceinline__ void read_choice(const DecodeExperts& p, Chosen* c) {
 }
 
 // act[slot][j] = silu(gate_j . h) * (up_j . h): a row pair is (gate_j, up_j) of one chosen expert
-__global__ void __launch_bounds__(DL_THREADS) decode_gate_up_kernel(const DecodeExperts p, int ks, int padded) {
+__global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const DecodeExperts p, int ks, int padded) {
   extern __shared__ __align__(16) uint8_t dg_smem[];  // weight rings, input, part[]
   __shared__ Chosen ch;
   float* xs = reinterpret_cast<float*>(dg_smem + DL_WARPS * DL_RING);
@@ -755,7 +819,7 @@ __global__ void __launch_bounds__(DL_THREADS) decode_gate_up_kernel(const Decode
 
 // out[n] = sum over the chosen experts of weight * (down_n . act) + (identity weights) * h[n]: the experts' vectors,
 // already multiplied by their weights, stand one after the other in shared memory
-__global__ void __launch_bounds__(DL_THREADS) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded) {
+__global__ void __launch_bounds__(DL_THREADS, 2) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded) {
   extern __shared__ __align__(16) uint8_t dd_smem[];  // weight rings, inputs [top][ff_padded], part[]
   __shared__ Chosen ch;
   float* xs = reinterpret_cast<float*>(dd_smem + DL_WARPS * DL_RING);
