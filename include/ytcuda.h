@@ -383,9 +383,10 @@ int ytcuda_window_attn_fwd(int dtype, const void* q, const void* k, const void* 
                            const int64_t* k_strides, const int64_t* v_strides, const int64_t* o_strides, int64_t pos0,
                            int window, int ring, float scale, float softcap, void* stream);
 
-/* Router of a mixture of experts with `identity` identity experts behind the `experts` real ones: s = softmax(logits)
- * over all of them, choice scores s + correction; of `groups` equal groups of neighbours only the `keep` whose largest
- * choice score is best can be chosen; the `top` largest choice scores are, with weights s (not renormalised).
+/* Router of a mixture of experts with `identity` pass-through experts behind the `experts` real ones: s = softmax(logits)
+ * over both kinds is the weight of a route (used as it is), s + correction its selection score. The routes are split into
+ * `groups` contiguous blocks of one size, ranked by their maximal selection score; the `top` routes with the largest
+ * selection scores are taken from the `keep` leading blocks.
  * choice / weight [rows, top] in the order of choice (-1: none left); rank [rows, top]: running number of the token
  * among its expert's tokens; count [experts] is increased by the arrivals (the caller zeroes it). */
 int ytcuda_moe_route(const float* logits, int64_t row_stride, const float* correction, int64_t rows, int experts,

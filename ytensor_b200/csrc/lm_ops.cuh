@@ -136,9 +136,9 @@ struct AppendKv {
 int append_kv(const AppendKv& a, cudaStream_t st);
 
 // ---------------------------------------------------------------- mixture of experts
-// `experts` experts and `identity` identity experts share one router: s = softmax(logits), choice scores s +
-// correction, only the `keep` best of `count` equal groups of neighbours (group score: its largest choice score) can
-// be chosen, the `top` largest choice scores are, and their weights are s.
+// `experts` experts and `identity` pass-through experts share one router: s = softmax(logits) decides the weights,
+// s + correction the selection. The routes are split into `count` contiguous blocks of one size, ranked by their maximal
+// selection score; the `top` routes are taken from the `keep` leading blocks.
 struct RouterSpec {
   int experts = 0, identity = 0, top = 0, count = 1, keep = 1;
 };
