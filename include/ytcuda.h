@@ -384,26 +384,64 @@ int ytcuda_window_attn_fwd(int dtype, const void* q, const void* k, const void* 
                            int window, int ring, float scale, float softcap, void* stream);
 
 /* Router of a mixture of experts with `identity` pass-through experts behind the `experts` real ones: s = softmax(logits)
- * over both kinds is the weight of a route (used as it is), s + correction its selection score. The routes are split into
+ * over both kinds (score 0) or sigmoid of every logit (score 1) is the weight of a route (used as it is), s + correction
+ * (NULL: s) its selection score. The routes are split into
  * `groups` contiguous blocks of one size, ranked by their maximal selection score; the `top` routes with the largest
  * selection scores are taken from the `keep` leading blocks.
  * choice / weight [rows, top] in the order of choice (-1: none left); rank [rows, top]: running number of the token
  * among its expert's tokens; count [experts] is increased by the arrivals (the caller zeroes it). */
 int ytcuda_moe_route(const float* logits, int64_t row_stride, const float* correction, int64_t rows, int experts,
-                     int identity, int top, int groups, int keep, int32_t* choice, float* weight, int32_t* rank,
+                     int identity, int top, int groups, int keep, int score, int32_t* choice, float* weight, int32_t* rank,
                      int32_t* count, void* stream);
 
 /* Residual stream around a sublayer: x += y / rms(y) * w_post (skipped when w_post is NULL), then
- * h = x / rms(x) * w_pre in fp32 or bf16 (skipped when w_pre is NULL); rms(v) = sqrt(mean(v^2) + eps) over the first
+ * h = x / rms(x) * w_pre in fp32 or bf16 (w_pre NULL: h = x; skipped when h is NULL); rms(v) = sqrt(mean(v^2) + eps) over the first
  * `width` of row_stride channels. One launch. */
 int ytcuda_residual_norm(float* x, const float* y, const float* w_post, const float* w_pre, void* h, int dtype, int64_t rows,
                          int width, int row_stride, float eps, void* stream);
 
 /* y[m, n] = act(x[m, k] . W[n, k]^T), W bf16, x and y bf16 (tensor cores) or fp32 (FFMA). act 0: none, 1: exact (erf)
- * gelu, 2: the rows of W alternate gate_j, up_j and y[m, n / 2] = silu(gate) * up. With block_group, rows come in blocks
- * of 128 and block i uses matrix block_group[i] of `groups` stacked ones (-1: the block is passed over). */
+ * gelu, 2: the rows of W alternate gate_j, up_j and y[m, n / 2] = silu(gate) * up, 3: max(z, 0)^2, 4: silu in the first
+ * act_cols columns, 5: alternating rows with g = min(gate, limit), u = up bounded to [-limit, limit], y[m, n / 2] =
+ * g sigmoid(1.702 g) (u + 1). With block_group, rows come in blocks of 128 and block i uses matrix block_group[i] of
+ * `groups` stacked ones (-1: the block is passed over). */
 int ytcuda_linear_act(int dtype, int act, const void* x, int64_t x_row_stride, const void* w_bf16, void* y,
-                      int64_t y_row_stride, int m, int n, int k, const int32_t* block_group, int groups, void* stream);
+                      int64_t y_row_stride, int m, int n, int k, int act_cols, float limit, const int32_t* block_group,
+                      int groups, void* stream);
+
+/* out = in / rms(in) * w * sigmoid(gate) row by row (w NULL: in * sigmoid(gate)); rms over the first `width` of `cols`
+ * channels (the others zero); strides in elements. */
+int ytcuda_gated_rows(int dtype, const void* in, int64_t in_stride, const void* gate, int64_t gate_stride, void* out,
+                      int64_t out_stride, int64_t rows, int cols, int width, const float* w, float eps, void* stream);
+
+/* Linear attention with a decayed state: per sequence and head S <- decay S + k v^T, o = S^T q, token by token. q, k
+ * [batch, len, heads, dim] and v [batch, len, heads, vdim] with rows of `ld` elements, o [batch, len, heads, vdim], state
+ * [batch, heads, dim, vdim] fp32 (read unless `first`, then written), decay [heads] fp32. path 0: automatic, 1: token by
+ * token, 2: chunks of 128 tokens on tcgen05 (bf16, dim = vdim = 128; YTC_UNSUPPORTED elsewhere). */
+int ytcuda_decayed_attn_fwd(int dtype, const void* q, const void* k, const void* v, int64_t ld, void* o, float* state,
+                            const float* decay, int batch, int len, int heads, int dim, int vdim, int first, int path,
+                            void* stream);
+
+/* Attention of batch * len query rows (at positions pos0 ..) over a cache of latents [batch, cap, rank + rot]: a row holds
+ * the normed latent c and a rotated key part r shared by the heads. Per head the key is [uk c, r], the value uv c. q
+ * [batch * len, heads, dim + rot] not yet rotated: dimensions 2 i and 2 i + 1 of its last `rot` turn by position * freq[i],
+ * i < rot / 2. uk [heads * dim, rank], uv [heads * vdim, rank] bf16; out [batch * len, heads, vdim]. The form for few rows. */
+int ytcuda_latent_attn_fwd(int dtype, const void* q, const void* uk_bf16, const void* uv_bf16, const void* cache, int64_t cap,
+                           void* out, int batch, int len, int64_t pos0, int heads, int dim, int rot, int vdim, int rank,
+                           const float* freq, float scale, void* stream);
+
+/* ---------------------------------------------------------------- handles of the models below */
+void ytcuda_lm_destroy(void* handle);
+/* Starts every sequence anew. */
+int ytcuda_lm_reset(void* handle);
+int64_t ytcuda_lm_cache_len(void* handle);
+/* One new token of a single sequence: 0 = the graph of fused decode kernels, 1 = one launch per operator as for longer
+ * inputs. */
+int ytcuda_lm_set_decode_path(void* handle, int path);
+/* Appends ids [batch, len] (device) to the sequences. want (HOST, n_want distinct row numbers in [0, batch * len), in
+ * the order of the tokens) selects the rows whose logits [n_want, vocab] (device, fp32) are computed. */
+int ytcuda_lm_forward(void* handle, const int32_t* ids, int len, const int32_t* want, int n_want, float* logits,
+                      void* stream);
 
 /* ---------------------------------------------------------------- Duzozen decoder
  * Decoder-only model: norm before and after each sublayer, sliding-window attention with capped scores, values mixed
@@ -432,21 +470,48 @@ typedef struct {
 } ytcuda_duzozen_layer;
 /* Returns NULL on an unsupported configuration (see ytcuda_last_error_string). */
 void* ytcuda_duzozen_create(const ytcuda_duzozen_config* cfg, const ytcuda_duzozen_layer* layers);
-void ytcuda_duzozen_destroy(void* handle);
 /* Registers a device weight (borrowed). "embed", "head" [vocab, width] bf16, "norm" [width] fp32; per layer fp32
  * "norm1", "norm1b", "norm2", "norm2b" [width], "vmix" [1], "correction" [experts + identity]; bf16 "qkv" [q heads, k
  * heads, v heads; width], "o" [width, heads * vdim], "up" / "down" [ff, width] / [width, ff] (dense) or [experts, 2 ff,
  * width] with gate_j, up_j alternating / [experts, width, ff], "router" [experts + identity, width]. */
 int ytcuda_duzozen_set_weight(void* handle, const char* name, int layer, const void* dptr);
-int ytcuda_duzozen_reset(void* handle);
-int64_t ytcuda_duzozen_cache_len(void* handle);
-/* One new token of a single sequence: 0 = the graph of fused decode kernels, 1 = one launch per operator as for longer
- * inputs. */
-int ytcuda_duzozen_set_decode_path(void* handle, int path);
-/* Appends ids [batch, len] (device) to the sequences. want (HOST, n_want distinct row numbers in [0, batch * len), in
- * the order of the tokens) selects the rows whose logits [n_want, vocab] (device, fp32) are computed. */
-int ytcuda_duzozen_forward(void* handle, const int32_t* ids, int len, const int32_t* want, int n_want, float* logits,
-                           void* stream);
+
+/* ---------------------------------------------------------------- Derupel decoder
+ * Decoder-only model: sublayers read the residual stream and are normed on their output only; linear attention with a
+ * decayed state or attention over cached latents, both with an output gate; dense (squared relu) feed-forward or a mixture
+ * of experts (bounded gates, sigmoid router that weighs the experts' inputs, shared expert). Sizes are padded by the caller
+ * (zero weights) to the stored sizes below; norms run over the *_width true channels. */
+#define YTC_MIXER_DECAYED 0
+#define YTC_MIXER_LATENT 1
+typedef struct {
+  int width, norm_width, vocab, layers;
+  int batch;      /* sequences, all of one length */
+  int max_tokens; /* longest sequence */
+  int chunk;      /* most tokens per sequence that run through the layers at once */
+  int dtype;      /* YTC_BF16: bf16 activations and cache, fp32 residual stream and state; YTC_F32: everything fp32 */
+  float eps;
+  float embed_scale;
+} ytcuda_derupel_config;
+typedef struct {
+  int mixer; /* YTC_MIXER_* */
+  int heads, dim, vdim;
+  int norm_width; /* YTC_MIXER_DECAYED: true channels of the concatenated heads */
+  int rot, rot_dims, head_ld, rank, q_rank, q_width, c_width; /* YTC_MIXER_LATENT; head_ld: elements per query head */
+  int mlp; /* YTC_MLP_* */
+  int ff, experts, top, shared_ff; /* shared_ff 0: no shared expert */
+  float scale;
+  float limit, shared_limit;
+} ytcuda_derupel_layer;
+/* Returns NULL on an unsupported configuration (see ytcuda_last_error_string). */
+void* ytcuda_derupel_create(const ytcuda_derupel_config* cfg, const ytcuda_derupel_layer* layers);
+/* Registers a device weight (borrowed). "embed", "head" [vocab, width] bf16, "norm" [width] fp32; per layer fp32 "norm1",
+ * "norm2" [width]; bf16 "in" [q heads, k heads, v heads, gate; width] or [query latent, latent, rotated key part, gate;
+ * width], "o" [width, heads * vdim]; fp32 "mix_norm" [heads * vdim], "decay" [heads]; fp32 "dq_norm" [q_rank], "dkv_norm"
+ * [rank], "freq" [rot_dims / 2]; bf16 "uq" [heads * head_ld, q_rank], "uk" [heads * dim, rank], "uv" [heads * vdim, rank],
+ * "expand" [heads * head_ld + heads * vdim, rank + rot] (per head uk and the identity over the rotated part, then uv);
+ * "up" / "down" [ff, width] / [width, ff] (dense) or [experts, 2 ff, width] with gate_j, up_j alternating / [experts,
+ * width, ff], "router" [experts, width], "shared_up" [2 shared_ff, width], "shared_down" [width, shared_ff]. */
+int ytcuda_derupel_set_weight(void* handle, const char* name, int layer, const void* dptr);
 
 #ifdef __cplusplus
 }

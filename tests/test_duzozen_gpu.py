@@ -136,7 +136,7 @@ def test_router(D, experts, identity, top, count, keep):
     rk, w = torch.empty_like(ch), torch.empty(rows, top, device="cuda")
     cnt = torch.zeros(experts, dtype=torch.int32, device="cuda")
     zd, cd = dev(z), dev(corr)
-    _lib.check(_lib.lib().ytcuda_moe_route(zd.data_ptr(), n, cd.data_ptr(), rows, experts, identity, top, count, keep,
+    _lib.check(_lib.lib().ytcuda_moe_route(zd.data_ptr(), n, cd.data_ptr(), rows, experts, identity, top, count, keep, 0,
                                            ch.data_ptr(), w.data_ptr(), rk.data_ptr(), cnt.data_ptr(), None))
     got, gw, grk = ch.cpu().numpy(), w.cpu().numpy(), rk.cpu().numpy()
     for t in range(rows):
@@ -184,7 +184,7 @@ def test_linear_with_activation(D, dtype, m, n, k):
     for act, want in ((0, z), (1, P.gelu_erf(z)), (2, P.silu(z[:, ::2]) * z[:, 1::2])):
         y = torch.empty(m, want.shape[1], dtype=tt, device="cuda")
         _lib.check(_lib.lib().ytcuda_linear_act(code, act, x.data_ptr(), k, w.data_ptr(), y.data_ptr(), want.shape[1], m, n, k,
-                                                None, 1, torch.cuda.current_stream().cuda_stream))
+                                                0, 0.0, None, 1, torch.cuda.current_stream().cuda_stream))
         assert normwise(y.float().cpu().numpy(), want) < (2e-6 if dtype == "float32" else 5e-3)
 
 
@@ -202,7 +202,7 @@ def test_grouped_linear(D, dtype):
         cols = n // 2 if act == 2 else n
         y = torch.full((m, cols), 7.0, dtype=tt, device="cuda")
         _lib.check(_lib.lib().ytcuda_linear_act(code, act, x.data_ptr(), k, w.data_ptr(), y.data_ptr(), cols, m, n, k,
-                                                bg.data_ptr(), E, torch.cuda.current_stream().cuda_stream))
+                                                0, 0.0, bg.data_ptr(), E, torch.cuda.current_stream().cuda_stream))
         got = y.float().cpu().numpy()
         for i, e in enumerate(blocks):
             rows = slice(128 * i, 128 * i + 128)

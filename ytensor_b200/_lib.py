@@ -75,16 +75,21 @@ SIGNATURES = {
     "ytcuda_qwen3_forward": (_i, [_vp, _vp, _i, _vp, _vp]),
     "ytcuda_window_attn_fwd": (_i, [_i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _i64, _i, _i, _f,
                                     _f, _vp]),
-    "ytcuda_moe_route": (_i, [_vp, _i64, _vp, _i64, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp]),
+    "ytcuda_moe_route": (_i, [_vp, _i64, _vp, _i64] + [_i] * 6 + [_vp, _vp, _vp, _vp, _vp]),
     "ytcuda_residual_norm": (_i, [_vp, _vp, _vp, _vp, _vp, _i, _i64, _i, _i, _f, _vp]),
-    "ytcuda_linear_act": (_i, [_i, _i, _vp, _i64, _vp, _vp, _i64, _i, _i, _i, _vp, _i, _vp]),
+    "ytcuda_linear_act": (_i, [_i, _i, _vp, _i64, _vp, _vp, _i64, _i, _i, _i, _i, _f, _vp, _i, _vp]),
+    "ytcuda_gated_rows": (_i, [_i, _vp, _i64, _vp, _i64, _vp, _i64, _i64, _i, _i, _vp, _f, _vp]),
+    "ytcuda_decayed_attn_fwd": (_i, [_i, _vp, _vp, _vp, _i64, _vp, _vp, _vp] + [_i] * 7 + [_vp]),
+    "ytcuda_latent_attn_fwd": (_i, [_i, _vp, _vp, _vp, _vp, _i64, _vp, _i, _i, _i64] + [_i] * 5 + [_vp, _f, _vp]),
+    "ytcuda_lm_destroy": (None, [_vp]),
+    "ytcuda_lm_reset": (_i, [_vp]),
+    "ytcuda_lm_cache_len": (_i64, [_vp]),
+    "ytcuda_lm_set_decode_path": (_i, [_vp, _i]),
+    "ytcuda_lm_forward": (_i, [_vp, _vp, _i, _vp, _i, _vp, _vp]),
     "ytcuda_duzozen_create": (_vp, [_vp, _vp]),
-    "ytcuda_duzozen_destroy": (None, [_vp]),
     "ytcuda_duzozen_set_weight": (_i, [_vp, C.c_char_p, _i, _vp]),
-    "ytcuda_duzozen_reset": (_i, [_vp]),
-    "ytcuda_duzozen_cache_len": (_i64, [_vp]),
-    "ytcuda_duzozen_set_decode_path": (_i, [_vp, _i]),
-    "ytcuda_duzozen_forward": (_i, [_vp, _vp, _i, _vp, _i, _vp, _vp]),
+    "ytcuda_derupel_create": (_vp, [_vp, _vp]),
+    "ytcuda_derupel_set_weight": (_i, [_vp, C.c_char_p, _i, _vp]),
 }
 
 

@@ -43,6 +43,8 @@ struct GemmTcParams {
   const uint8_t* tile_live;
   // linear layers of the language models (LinearEpilogue, lm_ops.cuh)
   int epi;                 // EPI_NONE: the store rules above; otherwise tc_store_epilogue
+  int act_cols;            // EPI_SILU
+  float limit, alpha_gate, shift;  // EPI_CLAMP_PAIRS
   // grouped product: every 128-row block of A belongs to one group (expert) or to none (-1, passed over); group g
   // multiplies rows g * group_rows .. of the stacked B operand. NULL = ordinary product.
   const int* tile_group;
@@ -135,18 +137,28 @@ __device__ __forceinline__ void tc_store_chunk(const GemmTcParams& p, const uint
   }
 }
 
+__device__ __forceinline__ float tc_clamped_gate(const GemmTcParams& p, float gate, float up) {
+  const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
+  return __fdividef(g, 1.f + __expf(-p.alpha_gate * g)) * (u + p.shift);
+}
 // Store with a fused activation and round-to-nearest-even narrowing (see LinearEpilogue). One thread holds 32
-// consecutive columns of one row; EPI_SWIGLU_PAIRS makes 16 results of them.
+// consecutive columns of one row; the gated pairs make 16 results of them.
 __device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const uint32_t (&r)[32], int64_t row_off, int gn0,
                                                   bool row_ok) {
   if (!row_ok) return;
-  if (p.epi == EPI_SWIGLU_PAIRS) {
+  if (p.epi == EPI_SWIGLU_PAIRS || p.epi == EPI_CLAMP_PAIRS) {
     uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + (gn0 >> 1);
     uint32_t w[8];
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const float a = lm_silu_fast(__uint_as_float(r[4 * j])) * __uint_as_float(r[4 * j + 1]);
-      const float b = lm_silu_fast(__uint_as_float(r[4 * j + 2])) * __uint_as_float(r[4 * j + 3]);
+      float a, b;
+      if (p.epi == EPI_SWIGLU_PAIRS) {
+        a = lm_silu_fast(__uint_as_float(r[4 * j])) * __uint_as_float(r[4 * j + 1]);
+        b = lm_silu_fast(__uint_as_float(r[4 * j + 2])) * __uint_as_float(r[4 * j + 3]);
+      } else {
+        a = tc_clamped_gate(p, __uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]));
+        b = tc_clamped_gate(p, __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
+      }
       w[j] = pack_bf16x2_rn(a, b);
     }
     if (gn0 + 32 <= p.N && (reinterpret_cast<uint64_t>(dst) & 15u) == 0) {
@@ -167,6 +179,12 @@ __device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const u
     if (p.epi == EPI_GELU_ERF) {
       a = lm_gelu_erf(a);
       b = lm_gelu_erf(b);
+    } else if (p.epi == EPI_RELU2) {
+      a = lm_relu2(a);
+      b = lm_relu2(b);
+    } else if (p.epi == EPI_SILU) {
+      if (gn0 + 2 * j < p.act_cols) a = lm_silu_fast(a);
+      if (gn0 + 2 * j + 1 < p.act_cols) b = lm_silu_fast(b);
     }
     w[j] = pack_bf16x2_rn(a, b);
   }
@@ -916,7 +934,10 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
   p.a_prefetch = g_tc_a_prefetch;
   p.split_loads = g_tc_split_loads;
   p.tile_live = nullptr;
-  p.epi = ex ? ex->epi : EPI_NONE;
+  const LinearEpilogue none, *e = ex ? ex : &none;
+  p.epi = e->epi;
+  p.act_cols = e->act_cols;
+  p.limit = e->limit; p.alpha_gate = e->alpha; p.shift = e->shift;
   p.tile_group = grouped ? ex->tile_group : nullptr;
   p.group_rows = n;
   p.status = device_status_word();
@@ -970,7 +991,7 @@ int linear_tc(const void* x, int64_t ldx, const void* w, int64_t ldw, void* y, i
   YTC_REQUIRE(tc_operand_ok(x, ldx, 1, 0, 1, m, k, &unused) && tc_operand_ok(w, ldw, 1, 0, 1, n, k, &unused),
               "linear_tc: operand rows must be 16-byte aligned");
   YTC_REQUIRE(ex.epi == EPI_NONE || out_dtype == YTC_BF16, "linear_tc: fused epilogues store bf16");
-  YTC_REQUIRE(ex.epi != EPI_SWIGLU_PAIRS || n % 2 == 0, "linear_tc: an odd number of gate / up rows");
+  YTC_REQUIRE(!epi_pairs(ex.epi) || n % 2 == 0, "linear_tc: an odd number of gate / up rows");
   YTC_REQUIRE(!ex.tile_group || m % TC_BM == 0, "linear_tc: grouped rows come in blocks of %d", TC_BM);
   return launch_tc(YTC_BF16, out_dtype, x, w, y, m, n, k, 1.f, 0.f, 0, ldx, 0, ldw, ldy, 1, 1, 0, 0, 0, st, &ex);
 }

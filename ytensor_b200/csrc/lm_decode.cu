@@ -1,4 +1,4 @@
-// One new token of a windowed language model: the kernels of a decode step.
+// One new token of a language model: the kernels of a decode step that the models share.
 //
 // A step is a chain of short kernels (projection with the norms before it, attention, projection, ...) queued as
 // programmatic dependent launches inside a CUDA graph. Every kernel requests what does not depend on the kernel in
@@ -55,22 +55,26 @@ __device__ __forceinline__ int staged_at(int c) { return (c & ~255) + ((c & 4) <
 
 struct InputSmem {  // shared memory of a staged input
   float* h;         // [padded] the vector, in staged order
-  float *x, *g_post, *g_pre;  // [k] residual row and norm weights (kind 2: unused)
+  float *x, *g_post, *g_pre;  // [k] residual row and norm weights (DECODE_GATED: g_post is the gate, no x)
 };
-static int input_floats(int kind, int k, int padded) { return padded + (kind == 2 ? 0 : 3 * k); }
-__device__ __forceinline__ InputSmem input_smem(float* p, int k, int padded) {
+__host__ __device__ __forceinline__ int input_floats(int kind, int k, int padded) {
+  return padded + (kind == DECODE_PLAIN ? 0 : kind == DECODE_GATED ? 2 * k : 3 * k);
+}
+__device__ __forceinline__ InputSmem input_smem(int kind, float* p, int k, int padded) {
+  if (kind == DECODE_GATED) return InputSmem{p, nullptr, p + padded, p + padded + k};
   return InputSmem{p, p + padded, p + padded + k, p + padded + 2 * k};
 }
 
 // Requests what the input needs besides the output of the kernel before (one copy group).
 __device__ __forceinline__ void prefetch_input(const DecodeInput& in, int k, const InputSmem& s) {
-  if (in.kind != 2)
+  if (in.kind != DECODE_PLAIN)
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
-      cp_async16(s.g_pre + c, in.w_pre + c);
-      if (in.kind == 1) {
+      if (in.w_pre) cp_async16(s.g_pre + c, in.w_pre + c);
+      if (in.kind == DECODE_RESIDUAL) {
         cp_async16(s.g_post + c, in.w_post + c);
         cp_async16(s.x + c, in.x_in + c);
       }
+      if (in.kind == DECODE_GATED && in.gate) cp_async16(s.g_post + c, in.gate + c);  // (written two kernels ago)
     }
   cp_async_commit();
 }
@@ -82,21 +86,45 @@ __device__ __forceinline__ void stage_input(const DecodeInput& in, int k, int pa
                                             bool writer, float* h_out) {
   for (int c = k + threadIdx.x * 4; c < padded; c += DL_THREADS * 4)
     *reinterpret_cast<float4*>(s.h + staged_at(c)) = make_float4(0.f, 0.f, 0.f, 0.f);
-  if (in.kind == 2) {
+  if (in.kind == DECODE_PLAIN) {
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4)
       *reinterpret_cast<float4*>(s.h + staged_at(c)) = *reinterpret_cast<const float4*>(in.plain + c);
     __syncthreads();
     return;
   }
   float ss = 0.f;
-  if (in.kind == 0) {
+  if (in.kind == DECODE_GATED) {
+    for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(in.plain + c);
+      *reinterpret_cast<float4*>(s.h + staged_at(c)) = v;
+      ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
+    }
+    const float inv = in.w_pre ? 1.0f / sqrtf(dl_block_sum(ss, red) / in.width + in.eps) : 1.f;
+    cp_async_wait<OLDER>();
+    for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
+      float4 v = *reinterpret_cast<const float4*>(s.h + staged_at(c));
+      if (in.w_pre) {
+        const float4 g = *reinterpret_cast<const float4*>(s.g_pre + c);
+        v.x *= inv * g.x; v.y *= inv * g.y; v.z *= inv * g.z; v.w *= inv * g.w;
+      }
+      if (in.gate) {
+        const float4 g = *reinterpret_cast<const float4*>(s.g_post + c);
+        v.x *= lm_sigmoid(g.x); v.y *= lm_sigmoid(g.y); v.z *= lm_sigmoid(g.z); v.w *= lm_sigmoid(g.w);
+      }
+      *reinterpret_cast<float4*>(s.h + staged_at(c)) = v;
+    }
+    __syncthreads();
+    return;
+  }
+  if (in.kind == DECODE_EMBED) {
     int id = *in.id;
     id = id < 0 ? 0 : (id >= in.vocab ? in.vocab - 1 : id);
     const uint16_t* row = in.embed + static_cast<int64_t>(id) * k;
     for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
       const uint2 u = *reinterpret_cast<const uint2*>(row + c);
-      const float4 x = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u),
-                                   __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+      const float e = in.embed_scale;
+      const float4 x = make_float4(e * __uint_as_float(u.x << 16), e * __uint_as_float(u.x & 0xFFFF0000u),
+                                   e * __uint_as_float(u.y << 16), e * __uint_as_float(u.y & 0xFFFF0000u));
       *reinterpret_cast<float4*>(s.x + c) = x;  // (every thread reads back its own columns only)
       if (writer) *reinterpret_cast<float4*>(in.x_out + c) = x;
     }
@@ -116,6 +144,15 @@ __device__ __forceinline__ void stage_input(const DecodeInput& in, int k, int pa
       *reinterpret_cast<float4*>(s.x + c) = x;
       if (writer) *reinterpret_cast<float4*>(in.x_out + c) = x;
     }
+  }
+  if (!in.w_pre) {
+    for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
+      const float4 x = *reinterpret_cast<const float4*>(s.x + c);
+      *reinterpret_cast<float4*>(s.h + staged_at(c)) = x;
+      if (writer && h_out) *reinterpret_cast<float4*>(h_out + c) = x;
+    }
+    __syncthreads();
+    return;
   }
   ss = 0.f;
   for (int c = threadIdx.x * 4; c < k; c += DL_THREADS * 4) {
@@ -243,7 +280,7 @@ static int dl_smem_check(const void* fn, int smem, const char* what) {
   return smem > 48 * 1024 ? ensure_dynamic_smem(fn, smem) : YTC_OK;
 }
 static int check_input(const DecodeInput& in, int k) {
-  YTC_REQUIRE(k > 0 && k % 8 == 0 && (in.kind == 2 || in.width <= k), "decode step: bad vector length %d", k);
+  YTC_REQUIRE(k > 0 && k % 8 == 0 && (in.kind == DECODE_PLAIN || in.width <= k), "decode step: bad vector length %d", k);
   return YTC_OK;
 }
 
@@ -251,8 +288,8 @@ static int check_input(const DecodeInput& in, int k) {
 __global__ void __launch_bounds__(DL_THREADS, 2) decode_linear_kernel(const DecodeLinear p, int ks, int padded) {
   extern __shared__ __align__(16) uint8_t dl_smem[];  // weight rings, input, part[]
   __shared__ float red[2 * DL_WARPS];
-  const InputSmem in = input_smem(reinterpret_cast<float*>(dl_smem + DL_WARPS * DL_RING), p.k, padded);
-  float* part = in.h + padded + (p.in.kind == 2 ? 0 : 3 * p.k);
+  const InputSmem in = input_smem(p.in.kind, reinterpret_cast<float*>(dl_smem + DL_WARPS * DL_RING), p.k, padded);
+  float* part = in.h + input_floats(p.in.kind, p.k, padded);
   int begin, end;
   my_pairs((p.n + 1) / 2, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
@@ -274,8 +311,7 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_linear_kernel(const Deco
   for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS) {
     const int row = begin * 2 + i;
     if (row >= p.n) continue;
-    const float v = sum_sub(part, i, ks);
-    p.out[row] = p.epi == EPI_GELU_ERF ? lm_gelu_erf(v) : v;
+    p.out[row] = lm_activation(p.ex, sum_sub(part, i, ks), row);
   }
   if (p.advance && blockIdx.x == 0 && threadIdx.x == 0) *p.advance += 1;
 }
@@ -649,20 +685,28 @@ __device__ __forceinline__ bool comes_before(float a, int i, float b, int j) { r
 __device__ __forceinline__ void block_route(float* s, float* c, float* g, float* red, const float* correction,
                                             const RouterSpec& r, int* choice, float* weight) {
   const int n = r.experts + r.identity;
-  float m = -INFINITY;
-  for (int i = threadIdx.x; i < n; i += DL_THREADS) m = fmaxf(m, s[i]);
-  m = block_max(m, red);
-  float sum = 0.f;
-  for (int i = threadIdx.x; i < n; i += DL_THREADS) {
-    const float e = expf(s[i] - m);
-    s[i] = e;
-    sum += e;
-  }
-  sum = dl_block_sum(sum, red + DL_WARPS);
-  for (int i = threadIdx.x; i < n; i += DL_THREADS) {
-    const float p = s[i] / sum;
-    s[i] = p;
-    c[i] = p + correction[i];
+  if (r.score == ROUTE_SIGMOID) {
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+      const float p = lm_sigmoid(s[i]);
+      s[i] = p;
+      c[i] = p + correction[i];
+    }
+  } else {
+    float m = -INFINITY;
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) m = fmaxf(m, s[i]);
+    m = block_max(m, red);
+    float sum = 0.f;
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+      const float e = expf(s[i] - m);
+      s[i] = e;
+      sum += e;
+    }
+    sum = dl_block_sum(sum, red + DL_WARPS);
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) {
+      const float p = s[i] / sum;
+      s[i] = p;
+      c[i] = p + correction[i];
+    }
   }
   if (threadIdx.x < r.top) {  // (places that no route takes)
     choice[threadIdx.x] = -1;
@@ -702,8 +746,8 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const Decod
   extern __shared__ __align__(16) uint8_t dr_smem[];  // weight rings, input, part[], scores[n], choice scores[n], groups
   __shared__ float red[2 * DL_WARPS];
   const int n = p.r.experts + p.r.identity, pairs = (n + 1) / 2;
-  const InputSmem in = input_smem(reinterpret_cast<float*>(dr_smem + DL_WARPS * DL_RING), p.k, padded);
-  float* part = in.h + padded + 3 * p.k;
+  const InputSmem in = input_smem(p.in.kind, reinterpret_cast<float*>(dr_smem + DL_WARPS * DL_RING), p.k, padded);
+  float* part = in.h + input_floats(p.in.kind, p.k, padded);
   float* s = part + ((pairs + DR_CLUSTER - 1) / DR_CLUSTER) * 2 * ks;
   float* c = s + n;
   float* g = c + n;
@@ -723,7 +767,7 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const Decod
   rp.start();
   float* corr = g + p.r.count;
   if (rank == 0)
-    for (int i = threadIdx.x; i < n; i += DL_THREADS) corr[i] = p.correction[i];
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) corr[i] = p.correction ? p.correction[i] : 0.f;
   asm volatile("barrier.cluster.arrive.relaxed.aligned;" ::: "memory");  // (this CTA has started)
   dependent_wait();
   dependent_trigger();
@@ -745,7 +789,7 @@ int decode_route(const DecodeRoute& a, cudaStream_t st) {
   const int ks = pick_ks(per, pieces);
   const int smem = DL_WARPS * DL_RING +
                    (input_floats(a.in.kind, a.k, padded) + per * 2 * ks + 3 * n + a.r.count) * static_cast<int>(sizeof(float));
-  YTC_REQUIRE(a.in.kind != 2, "decode step: the router's input is a normed residual row");
+  YTC_REQUIRE(a.in.kind == DECODE_EMBED || a.in.kind == DECODE_RESIDUAL, "decode step: the router's input is a normed residual row");
   if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_route_kernel), smem, "the router")) != YTC_OK) return s;
   YTC_CUDA(launch_cluster(decode_route_kernel, DR_CLUSTER, DR_CLUSTER, smem, st, a, ks, padded));
   count_launch();
@@ -785,7 +829,8 @@ __device__ __forceinline__ void read_choice(const DecodeExperts& p, Chosen* c) {
   __syncthreads();
 }
 
-// act[slot][j] = silu(gate_j . h) * (up_j . h): a row pair is (gate_j, up_j) of one chosen expert
+// mid[slot][j] = gated(gate_j . h, up_j . h): a row pair is (gate_j, up_j) of one chosen expert, the shared expert's pairs
+// come first
 __global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const DecodeExperts p, int ks, int padded) {
   extern __shared__ __align__(16) uint8_t dg_smem[];  // weight rings, input, part[]
   __shared__ Chosen ch;
@@ -795,12 +840,17 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const Dec
   dependent_trigger();
   read_choice(p, &ch);
   int begin, end;
-  my_pairs(ch.n * p.ff, begin, end);
+  my_pairs(p.shared_ff + ch.n * p.ff, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
   auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
-    const int col = piece * DL_PIECE + lane8, i = pair / p.ff, j = pair - i * p.ff;
+    const int col = piece * DL_PIECE + lane8;
     ok0 = ok1 = col < p.k;
-    p0 = p.gate_up + (static_cast<int64_t>(ch.expert[i]) * 2 * p.ff + 2 * j) * p.k + (ok0 ? col : 0);
+    if (pair < p.shared_ff) {
+      p0 = p.shared_gate_up + static_cast<int64_t>(2 * pair) * p.k + (ok0 ? col : 0);
+    } else {
+      const int q = pair - p.shared_ff, i = q / p.ff, j = q - i * p.ff;
+      p0 = p.gate_up + (static_cast<int64_t>(ch.expert[i]) * 2 * p.ff + 2 * j) * p.k + (ok0 ? col : 0);
+    }
     p1 = p0 + p.k;
   };
   RowPairs<decltype(addr)> rp(addr, dg_smem, begin, end, (p.k + DL_PIECE - 1) / DL_PIECE, ks);
@@ -812,43 +862,63 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_gate_up_kernel(const Dec
   rp.run(xs, part);
   __syncthreads();
   for (int i = threadIdx.x; i < end - begin; i += DL_THREADS) {
-    const int pair = begin + i, e = pair / p.ff, j = pair - e * p.ff;
-    p.act[static_cast<int64_t>(ch.slot[e]) * p.ff + j] = lm_silu(sum_sub(part, 2 * i, ks)) * sum_sub(part, 2 * i + 1, ks);
+    const int pair = begin + i;
+    const float g = sum_sub(part, 2 * i, ks), u = sum_sub(part, 2 * i + 1, ks);
+    if (pair < p.shared_ff) {
+      p.mid[static_cast<int64_t>(p.r.top) * p.ff + pair] = lm_gated(p.shared_act, g, u);
+    } else {
+      const int q = pair - p.shared_ff, e = q / p.ff, j = q - e * p.ff;
+      const float w = p.scale_input ? ch.weight[e] : 1.f;  // (both products are linear in the expert's input)
+      p.mid[static_cast<int64_t>(ch.slot[e]) * p.ff + j] = lm_gated(p.act, w * g, w * u);
+    }
   }
 }
 
-// out[n] = sum over the chosen experts of weight * (down_n . act) + (identity weights) * h[n]: the experts' vectors,
-// already multiplied by their weights, stand one after the other in shared memory
-__global__ void __launch_bounds__(DL_THREADS, 2) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded) {
-  extern __shared__ __align__(16) uint8_t dd_smem[];  // weight rings, inputs [top][ff_padded], part[]
+// out[n] = sum over the chosen experts of weight * (down_n . mid) + (identity weights) * h[n] + (shared down_n . mid): the
+// experts' vectors, already multiplied by their weights, stand one after the other in shared memory, the shared one first
+__global__ void __launch_bounds__(DL_THREADS, 2) decode_down_kernel(const DecodeExperts p, int ks, int ff_padded,
+                                                                    int shared_padded) {
+  extern __shared__ __align__(16) uint8_t dd_smem[];  // weight rings, inputs [shared_padded], [top][ff_padded], part[]
   __shared__ Chosen ch;
   float* xs = reinterpret_cast<float*>(dd_smem + DL_WARPS * DL_RING);
-  float* part = xs + p.r.top * ff_padded;
+  float* part = xs + shared_padded + p.r.top * ff_padded;
   // (the choice was made two kernels ago: the kernel before this one has already waited for it)
   read_choice(p, &ch);
   int begin, end;
   my_pairs(p.k / 2, begin, end);
   const int lane8 = (threadIdx.x & 31) * 8;
-  const int per_expert = ff_padded / DL_PIECE;
+  const int per_expert = ff_padded / DL_PIECE, shared_pieces = shared_padded / DL_PIECE;
   auto addr = [&](int pair, int piece, const uint16_t*& p0, const uint16_t*& p1, bool& ok0, bool& ok1) {
-    const int i = piece / per_expert, col = (piece - i * per_expert) * DL_PIECE + lane8;
+    if (piece < shared_pieces) {
+      const int col = piece * DL_PIECE + lane8;
+      ok0 = ok1 = col < p.shared_ff;
+      p0 = p.shared_down + static_cast<int64_t>(2 * pair) * p.shared_ff + (ok0 ? col : 0);
+      p1 = p0 + p.shared_ff;
+      return;
+    }
+    const int q = piece - shared_pieces, i = q / per_expert, col = (q - i * per_expert) * DL_PIECE + lane8;
     ok0 = ok1 = col < p.ff;
     p0 = p.down + (static_cast<int64_t>(ch.expert[i]) * p.k + 2 * pair) * p.ff + (ok0 ? col : 0);
     p1 = p0 + p.ff;
   };
-  const int pieces = ch.n * per_expert;
+  const int pieces = shared_pieces + ch.n * per_expert;
   const int ks_here = pieces < ks ? 1 : ks;
   RowPairs<decltype(addr)> rp(addr, dd_smem, begin, pieces > 0 ? end : begin, pieces, ks_here);
   rp.start();
   dependent_wait();
   dependent_trigger();
+  for (int c = threadIdx.x * 4; c < shared_padded; c += DL_THREADS * 4)
+    *reinterpret_cast<float4*>(xs + staged_at(c)) =
+        c < p.shared_ff ? *reinterpret_cast<const float4*>(p.mid + static_cast<int64_t>(p.r.top) * p.ff + c)
+                        : make_float4(0.f, 0.f, 0.f, 0.f);
   const int per4 = ff_padded / 4;
   for (int v = threadIdx.x; v < ch.n * per4; v += DL_THREADS) {
     const int i = v / per4, c = (v - i * per4) * 4;
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < p.ff) a = *reinterpret_cast<const float4*>(p.act + static_cast<int64_t>(ch.slot[i]) * p.ff + c);
-    const float w = ch.weight[i];
-    *reinterpret_cast<float4*>(xs + i * ff_padded + staged_at(c)) = make_float4(w * a.x, w * a.y, w * a.z, w * a.w);
+    if (c < p.ff) a = *reinterpret_cast<const float4*>(p.mid + static_cast<int64_t>(ch.slot[i]) * p.ff + c);
+    const float w = p.scale_input ? 1.f : ch.weight[i];
+    *reinterpret_cast<float4*>(xs + shared_padded + i * ff_padded + staged_at(c)) =
+        make_float4(w * a.x, w * a.y, w * a.z, w * a.w);
   }
   __syncthreads();
   rp.run(xs, part);
@@ -860,10 +930,10 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_down_kernel(const Decode
 }
 
 int decode_experts(const DecodeExperts& a, cudaStream_t st) {
-  YTC_REQUIRE(a.k % 8 == 0 && a.ff % 8 == 0 && a.r.top <= LM_MAX_TOP, "decode step: bad expert size");
+  YTC_REQUIRE(a.k % 8 == 0 && a.ff % 8 == 0 && a.shared_ff % 8 == 0 && a.r.top <= LM_MAX_TOP, "decode step: bad expert size");
   int s;
   {
-    const int pieces = (a.k + DL_PIECE - 1) / DL_PIECE, padded = pieces * DL_PIECE, pairs = a.r.top * a.ff;
+    const int pieces = (a.k + DL_PIECE - 1) / DL_PIECE, padded = pieces * DL_PIECE, pairs = a.shared_ff + a.r.top * a.ff;
     const int grid = pairs < sm_count() ? pairs : sm_count();
     const int per = (pairs + grid - 1) / grid, ks = pick_ks(per, pieces);
     const int smem = DL_WARPS * DL_RING + (padded + per * 2 * ks) * static_cast<int>(sizeof(float));
@@ -873,11 +943,13 @@ int decode_experts(const DecodeExperts& a, cudaStream_t st) {
     YTC_CUDA(cudaGetLastError());
   }
   const int per_expert = (a.ff + DL_PIECE - 1) / DL_PIECE, ff_padded = per_expert * DL_PIECE, pairs = a.k / 2;
+  const int shared_padded = (a.shared_ff + DL_PIECE - 1) / DL_PIECE * DL_PIECE;
   const int grid = pairs < sm_count() ? pairs : sm_count();
-  const int per = (pairs + grid - 1) / grid, ks = pick_ks(per, a.r.top * per_expert);
-  const int smem = DL_WARPS * DL_RING + (a.r.top * ff_padded + per * 2 * ks) * static_cast<int>(sizeof(float));
+  const int per = (pairs + grid - 1) / grid, ks = pick_ks(per, a.r.top * per_expert + shared_padded / DL_PIECE);
+  const int smem = DL_WARPS * DL_RING +
+                   (shared_padded + a.r.top * ff_padded + per * 2 * ks) * static_cast<int>(sizeof(float));
   if ((s = dl_smem_check(reinterpret_cast<const void*>(decode_down_kernel), smem, "the experts' activations")) != YTC_OK) return s;
-  YTC_CUDA(launch_overlapped(decode_down_kernel, dim3(grid), dim3(DL_THREADS), smem, st, a, ks, ff_padded));
+  YTC_CUDA(launch_overlapped(decode_down_kernel, dim3(grid), dim3(DL_THREADS), smem, st, a, ks, ff_padded, shared_padded));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;

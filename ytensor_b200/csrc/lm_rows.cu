@@ -7,9 +7,9 @@
 namespace ytk {
 
 // ------------------------------------------------------------------ embedding gather
-// out[t, :] = float(table[ids[t], :])   (reference qwen3.cpp:378-385)
+// out[t, :] = scale * float(table[ids[t], :])   (scale 1: reference qwen3.cpp:378-385)
 __global__ void __launch_bounds__(256) embedding_kernel(const uint16_t* table, const int* ids, float* out, int64_t n,
-                                                        int hidden, int vocab) {
+                                                        int hidden, int vocab, float scale) {
   const int per_row = hidden / 4;
   const int64_t total = n * per_row;
   for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < total;
@@ -20,12 +20,22 @@ __global__ void __launch_bounds__(256) embedding_kernel(const uint16_t* table, c
     id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
     const uint2 w = *reinterpret_cast<const uint2*>(table + static_cast<int64_t>(id) * hidden + c);
     float4 o;
-    o.x = bf16_bits_to_f32(static_cast<uint16_t>(w.x & 0xFFFF));
-    o.y = bf16_bits_to_f32(static_cast<uint16_t>(w.x >> 16));
-    o.z = bf16_bits_to_f32(static_cast<uint16_t>(w.y & 0xFFFF));
-    o.w = bf16_bits_to_f32(static_cast<uint16_t>(w.y >> 16));
+    o.x = scale * bf16_bits_to_f32(static_cast<uint16_t>(w.x & 0xFFFF));
+    o.y = scale * bf16_bits_to_f32(static_cast<uint16_t>(w.x >> 16));
+    o.z = scale * bf16_bits_to_f32(static_cast<uint16_t>(w.y & 0xFFFF));
+    o.w = scale * bf16_bits_to_f32(static_cast<uint16_t>(w.y >> 16));
     *reinterpret_cast<float4*>(out + t * hidden + c) = o;
   }
+}
+
+int embed_rows(const uint16_t* table, const int* ids, float* x, int64_t rows, int width, int vocab, float scale,
+               cudaStream_t st) {
+  if (rows <= 0) return YTC_OK;
+  const int64_t blocks = (rows * (width / 4) + 255) / 256, cap = static_cast<int64_t>(sm_count()) * 16;
+  embedding_kernel<<<static_cast<unsigned>(blocks < cap ? blocks : cap), 256, 0, st>>>(table, ids, x, rows, width, vocab, scale);
+  count_launch();
+  YTC_CUDA(cudaGetLastError());
+  return YTC_OK;
 }
 
 // ------------------------------------------------------------------ residual stream
@@ -64,11 +74,14 @@ __global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const Residua
     if (p.slot) {
       if (threadIdx.x < p.top) {
         s_slot[threadIdx.x] = p.slot[row * p.top + threadIdx.x];
-        s_weight[threadIdx.x] = p.weight[row * p.top + threadIdx.x];
+        s_weight[threadIdx.x] = p.weight ? p.weight[row * p.top + threadIdx.x] : 1.f;
       }
       __syncthreads();
 #pragma unroll
-      for (int i = 0; i < VPT; ++i) yv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int i = 0; i < VPT; ++i) {
+        const int c = threadIdx.x + i * RN_THREADS;
+        yv[i] = p.y && c < nv ? reinterpret_cast<const float4*>(p.y + row * p.ld)[c] : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
       for (int k = 0; k < p.top; ++k) {  // in the order of choice: the sum does not depend on the batch
         const int s = s_slot[k];
         if (s < -1) continue;
@@ -115,7 +128,18 @@ __global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const Residua
       reinterpret_cast<float4*>(x)[c] = xv[i];
     }
   }
-  if (!p.w_pre) return;
+  if (!p.h) return;
+  T* h = static_cast<T*>(p.h) + static_cast<int64_t>(blockIdx.x) * p.ld;
+  if (!p.w_pre) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * RN_THREADS;
+      if (c >= nv) continue;
+      if (sizeof(T) == 4) reinterpret_cast<float4*>(h)[c] = xv[i];
+      else reinterpret_cast<uint2*>(h)[c] = make_uint2(pack_bf16x2_rn(xv[i].x, xv[i].y), pack_bf16x2_rn(xv[i].z, xv[i].w));
+    }
+    return;
+  }
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
@@ -123,7 +147,6 @@ __global__ void __launch_bounds__(RN_THREADS) residual_norm_kernel(const Residua
     ss = fmaf(xv[i].z, xv[i].z, ss); ss = fmaf(xv[i].w, xv[i].w, ss);
   }
   const float inv = 1.0f / sqrtf(rn_block_sum(ss, red[1]) / p.width + p.eps);
-  T* h = static_cast<T*>(p.h) + static_cast<int64_t>(blockIdx.x) * p.ld;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * RN_THREADS;
@@ -157,6 +180,73 @@ int residual_norm(const ResidualNorm& a, cudaStream_t st) {
   if (a.rows <= 0) return YTC_OK;
   YTC_REQUIRE(a.ld % 8 == 0 && a.width > 0 && a.width <= a.ld && a.top <= LM_MAX_TOP, "residual_norm: bad extent");
   return a.dtype == YTC_BF16 ? residual_norm_t<uint16_t>(a, st) : residual_norm_t<float>(a, st);
+}
+
+// ------------------------------------------------------------------ output gate
+// One row per CTA, pieces of 8 elements per thread; without a norm a row's pieces are independent.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(RN_THREADS) gated_rows_kernel(const GatedRows p) {
+  __shared__ float red[RN_THREADS / 32];
+  dependent_wait();
+  dependent_trigger();
+  const int64_t row = blockIdx.x;
+  const T* in = static_cast<const T*>(p.in) + row * p.ld_in;
+  const T* gate = static_cast<const T*>(p.gate) + row * p.ld_gate;
+  T* out = static_cast<T*>(p.out) + row * p.ld_out;
+  const int nv = p.cols / 8;
+  float f[VPT][8];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c >= nv) continue;
+    Vec8<T>::load(in + c * 8, f[i]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(f[i][e], f[i][e], ss);
+  }
+  float inv = 1.f;
+  if (p.w) inv = 1.0f / sqrtf(rn_block_sum(ss, red) / p.width + p.eps);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * RN_THREADS;
+    if (c >= nv) continue;
+    float g[8];
+    if (p.w) {
+      Vec8<float>::load(p.w + c * 8, g);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) f[i][e] *= inv * g[e];
+    }
+    Vec8<T>::load(gate + c * 8, g);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[i][e] *= sizeof(T) == 4 ? lm_sigmoid(g[e]) : lm_sigmoid_fast(g[e]);
+    Vec8<T>::store(out + c * 8, f[i]);
+  }
+}
+
+template <typename T>
+static int gated_rows_t(const GatedRows& a, cudaStream_t st) {
+  const int vpt = (a.cols / 8 + RN_THREADS - 1) / RN_THREADS;
+  void (*fn)(GatedRows) = nullptr;
+  if (vpt <= 1) fn = gated_rows_kernel<T, 1>;
+  else if (vpt <= 2) fn = gated_rows_kernel<T, 2>;
+  else if (vpt <= 4) fn = gated_rows_kernel<T, 4>;
+  else if (vpt <= 8) fn = gated_rows_kernel<T, 8>;
+  else {
+    set_last_error("gated_rows: rows of more than %d channels are not supported", 8 * 8 * RN_THREADS);
+    return YTC_UNSUPPORTED;
+  }
+  YTC_CUDA(launch_overlapped(fn, dim3(static_cast<unsigned>(a.rows)), dim3(RN_THREADS), 0, st, a));
+  count_launch();
+  YTC_CUDA(cudaGetLastError());
+  return YTC_OK;
+}
+
+int gated_rows(const GatedRows& a, cudaStream_t st) {
+  if (a.rows <= 0) return YTC_OK;
+  YTC_REQUIRE(a.cols > 0 && a.cols % 8 == 0 && a.ld_in % 8 == 0 && a.ld_gate % 8 == 0 && a.ld_out % 8 == 0 &&
+                  (!a.w || (a.width > 0 && a.width <= a.cols)),
+              "gated_rows: bad extent");
+  return a.dtype == YTC_BF16 ? gated_rows_t<uint16_t>(a, st) : gated_rows_t<float>(a, st);
 }
 
 // ------------------------------------------------------------------ K/V append
@@ -216,8 +306,8 @@ struct LinearF32Params {
   const uint16_t* w;
   float* y;
   int64_t ldx, ldw, ldy;
-  int m, n, k, epi;
-  const int* tile_group;
+  int m, n, k;
+  LinearEpilogue ex;
 };
 __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Params p) {
   __shared__ float xs[LF_BK][LF_BM + 4], ws[LF_BK][LF_BN + 4];
@@ -225,8 +315,8 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Params p
   dependent_trigger();
   const int m0 = blockIdx.y * LF_BM, n0 = blockIdx.x * LF_BN;
   int64_t w_row0 = 0;
-  if (p.tile_group) {
-    const int g = p.tile_group[m0 / LM_GROUP_ROWS];
+  if (p.ex.tile_group) {
+    const int g = p.ex.tile_group[m0 / LM_GROUP_ROWS];
     if (g < 0) return;
     w_row0 = static_cast<int64_t>(g) * p.n;
   }
@@ -259,18 +349,18 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const LinearF32Params p
   for (int i = 0; i < 4; ++i) {
     const int m = m0 + ty * 4 + i;
     if (m >= p.m) continue;
-    if (p.epi == EPI_SWIGLU_PAIRS) {
+    if (p.ex.epi == EPI_SWIGLU_PAIRS || p.ex.epi == EPI_CLAMP_PAIRS) {
 #pragma unroll
       for (int j = 0; j < 4; j += 2) {
         const int n = n0 + tx * 4 + j;
-        if (n + 1 < p.n) p.y[m * p.ldy + n / 2] = lm_silu(acc[i][j]) * acc[i][j + 1];
+        if (n + 1 < p.n) p.y[m * p.ldy + n / 2] = lm_gated(p.ex, acc[i][j], acc[i][j + 1]);
       }
       continue;
     }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int n = n0 + tx * 4 + j;
-      if (n < p.n) p.y[m * p.ldy + n] = p.epi == EPI_GELU_ERF ? lm_gelu_erf(acc[i][j]) : acc[i][j];
+      if (n < p.n) p.y[m * p.ldy + n] = lm_activation(p.ex, acc[i][j], n);
     }
   }
 }
@@ -279,10 +369,10 @@ int linear_f32(const float* x, int64_t ldx, const uint16_t* w, int64_t ldw, floa
                const LinearEpilogue& ex, cudaStream_t st) {
   if (m <= 0 || n <= 0) return YTC_OK;
   YTC_REQUIRE(k % 4 == 0 && ldx % 4 == 0 && ldw % 4 == 0, "linear_f32: rows must be whole groups of four elements");
-  YTC_REQUIRE(ex.epi != EPI_SWIGLU_PAIRS || n % 2 == 0, "linear_f32: an odd number of gate / up rows");
+  YTC_REQUIRE(!epi_pairs(ex.epi) || n % 2 == 0, "linear_f32: an odd number of gate / up rows");
   const int64_t tm = (static_cast<int64_t>(m) + LF_BM - 1) / LF_BM;
   YTC_REQUIRE(tm <= 65535, "linear_f32: too many rows");
-  LinearF32Params p{x, w, y, ldx, ldw, ldy, m, n, k, ex.epi, ex.tile_group};
+  LinearF32Params p{x, w, y, ldx, ldw, ldy, m, n, k, ex};
   YTC_CUDA(launch_overlapped(linear_f32_kernel, dim3((n + LF_BN - 1) / LF_BN, static_cast<unsigned>(tm)), dim3(256), 0, st, p));
   count_launch();
   YTC_CUDA(cudaGetLastError());
@@ -301,13 +391,8 @@ int ytcuda_embedding(const void* table_bf16, const int32_t* ids, float* out, int
   if (n == 0 || hidden == 0) return YTC_OK;
   YTC_REQUIRE(table_bf16 && ids && out, "ytcuda_embedding: null tensor");
   YTC_REQUIRE(hidden % 4 == 0, "ytcuda_embedding: hidden must be a multiple of 4");
-  const int64_t blocks = (n * (hidden / 4) + 255) / 256;
-  const int64_t cap = static_cast<int64_t>(sm_count()) * 16;
-  embedding_kernel<<<static_cast<unsigned>(blocks < cap ? blocks : cap), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const uint16_t*>(table_bf16), ids, out, n, hidden, vocab);
-  count_launch();
-  YTC_CUDA(cudaGetLastError());
-  return YTC_OK;
+  return embed_rows(static_cast<const uint16_t*>(table_bf16), ids, out, n, hidden, vocab, 1.f,
+                    static_cast<cudaStream_t>(stream));
 }
 
 }  // extern "C"

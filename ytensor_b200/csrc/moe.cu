@@ -53,14 +53,16 @@ int moe_route(const float* logits, int64_t ld, const float* correction, int64_t 
 
 constexpr int MG_THREADS = 256;
 
-__global__ void __launch_bounds__(MG_THREADS) moe_gather_kernel(const uint4* h, int row_vecs, int64_t rows,
-                                                                const RouterSpec r, const int* choice, const int* rank,
-                                                                const int* count, uint4* grouped, int* slot,
-                                                                int* tile_group, int n_tiles) {
+// T: float or bf16 bits (of scaled copies; a plain copy moves 16-byte vectors whatever they hold).
+template <typename T>
+__global__ void __launch_bounds__(MG_THREADS) moe_gather_kernel(const MoeGather p) {
   extern __shared__ int first_tile[];  // [experts + 1]: first block of every expert
   __shared__ int warp_sum[MG_THREADS / 32];
   dependent_wait();
   dependent_trigger();
+  const RouterSpec r = p.r;
+  const int *count = p.count, n_tiles = p.n_tiles;
+  int* tile_group = p.tile_group;
   // prefix sum of the blocks per expert, the same in every CTA
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   int carry = 0;
@@ -92,31 +94,45 @@ __global__ void __launch_bounds__(MG_THREADS) moe_gather_kernel(const uint4* h, 
     for (int e = threadIdx.x; e < r.experts; e += MG_THREADS)
       for (int t = first_tile[e]; t < first_tile[e + 1] && t < n_tiles; ++t) tile_group[t] = e;
   }
-  const int64_t pairs = rows * r.top;
+  const int64_t pairs = p.rows * r.top;
+  const int row_vecs = p.ld * static_cast<int>(sizeof(T)) / 16;
   // one warp per (token, choice)
   for (int64_t i = static_cast<int64_t>(blockIdx.x) * (MG_THREADS / 32) + warp; i < pairs;
        i += static_cast<int64_t>(gridDim.x) * (MG_THREADS / 32)) {
-    const int c = choice[i];
+    const int c = p.choice[i];
     const int64_t row = i / r.top;
     if (c < 0 || c >= r.experts) {
-      if (lane == 0) slot[i] = c < 0 ? -2 : -1;
+      if (lane == 0) p.slot[i] = c < 0 ? -2 : -1;
       continue;
     }
-    const int dst = first_tile[c] * LM_GROUP_ROWS + rank[i];
-    if (lane == 0) slot[i] = dst;
-    for (int v = lane; v < row_vecs; v += 32) grouped[static_cast<int64_t>(dst) * row_vecs + v] = h[row * row_vecs + v];
+    const int dst = first_tile[c] * LM_GROUP_ROWS + p.rank[i];
+    if (lane == 0) p.slot[i] = dst;
+    if (p.weight) {
+      const float w = p.weight[i];
+      const float* src = p.x + row * p.ld;
+      T* out = static_cast<T*>(p.grouped) + static_cast<int64_t>(dst) * p.ld;
+      for (int v = lane * 8; v < p.ld; v += 256) {
+        float f[8];
+        Vec8<float>::load(src + v, f);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) f[e] *= w;
+        Vec8<T>::store(out + v, f);
+      }
+    } else {
+      const uint4* src = static_cast<const uint4*>(p.h) + row * row_vecs;
+      uint4* out = static_cast<uint4*>(p.grouped) + static_cast<int64_t>(dst) * row_vecs;
+      for (int v = lane; v < row_vecs; v += 32) out[v] = src[v];
+    }
   }
 }
 
-int moe_gather(const void* h, int dtype, int ld, int64_t rows, const RouterSpec& r, const int* choice, const int* rank,
-               const int* count, void* grouped, int* slot, int* tile_group, int n_tiles, cudaStream_t st) {
-  YTC_REQUIRE(ld % 8 == 0 && n_tiles >= moe_max_tiles(rows, r), "moe_gather: bad extent");
-  if (rows <= 0) return YTC_OK;
-  const int row_vecs = ld * dtype_size(dtype) / 16;
-  const int64_t blocks = (rows * r.top + MG_THREADS / 32 - 1) / (MG_THREADS / 32), cap = static_cast<int64_t>(sm_count()) * 8;
-  YTC_CUDA(launch_overlapped(moe_gather_kernel, dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)), dim3(MG_THREADS),
-                             (r.experts + 1) * sizeof(int), st, static_cast<const uint4*>(h), row_vecs, rows, r, choice,
-                             rank, count, static_cast<uint4*>(grouped), slot, tile_group, n_tiles));
+int moe_gather(const MoeGather& g, cudaStream_t st) {
+  YTC_REQUIRE(g.ld % 8 == 0 && g.n_tiles >= moe_max_tiles(g.rows, g.r) && (!g.weight || g.x), "moe_gather: bad extent");
+  if (g.rows <= 0) return YTC_OK;
+  const int64_t blocks = (g.rows * g.r.top + MG_THREADS / 32 - 1) / (MG_THREADS / 32), cap = static_cast<int64_t>(sm_count()) * 8;
+  YTC_CUDA(launch_overlapped(g.dtype == YTC_BF16 ? moe_gather_kernel<uint16_t> : moe_gather_kernel<float>,
+                             dim3(static_cast<unsigned>(blocks < cap ? blocks : cap)), dim3(MG_THREADS),
+                             (g.r.experts + 1) * sizeof(int), st, g));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;

@@ -1,21 +1,15 @@
-"""Host side of the Duzozen language model: configuration, weights (padding, fusing, upload) and the wrapper over the
-model handle of the C ABI (ytcuda_duzozen_*).
+"""Host side of the Duzozen language model: configuration and weights (padding, fusing) for the model handle of the C ABI
+(ytcuda_duzozen_*; native_lm.py has what it shares with other models).
 
 The kernels want widths in multiples of 8 and, for the tensor-core attention, head dims of 64 or 128. Any other size is
 padded here with zero weights: padded channels of the residual stream, of a head or of a feed-forward stay zero, and
-norms run over the true width. torch is used for device memory only."""
+norms run over the true width."""
 from __future__ import annotations
 
 import ctypes as C
 from dataclasses import dataclass, field
 
-import numpy as np
-
-from . import _lib
-from ._lib import check, lib
-from .causal_lm import CausalLM
-
-MLP_NONE, MLP_DENSE, MLP_MOE = 0, 1, 2
+from .native_lm import MLP_DENSE, MLP_MOE, MLP_NONE, NativeLM, up8
 
 
 class _ConfigC(C.Structure):
@@ -127,154 +121,54 @@ class DuzozenConfig:
         return s
 
 
-def _up8(n: int) -> int:
-    return (n + 7) // 8 * 8
+class DuzozenForCausalLM(NativeLM):
+    """With `chunk`, a layer's window bounds its K/V ring."""
 
+    native = "duzozen"
 
-class DuzozenForCausalLM(CausalLM):
-    """Device model for `batch` sequences of up to `max_tokens` tokens. dtype "bfloat16": bf16 activations, cache and
-    tensor-core products, fp32 residual stream, norms, scores and router; "float32": everything fp32 (weights stay in
-    their bf16 storage, the products are the same numbers). chunk: most tokens per sequence that run through the layers
-    at once; with it a layer's window bounds its K/V ring."""
-
-    def __init__(self, cfg: DuzozenConfig, batch: int = 1, max_tokens: int = 4096, dtype: str = "bfloat16",
-                 chunk: int = 4096):
-        import torch
-        self.torch = torch
-        if dtype not in ("bfloat16", "float32"):
-            raise ValueError(f"dtype must be bfloat16 or float32, not {dtype}")
-        self.cfg, self.batch, self.dtype, self.max_tokens = cfg, batch, dtype, max_tokens
-        self.L = lib()
-        self.width_p = _up8(cfg.width)
-        dt = _lib.BF16 if dtype == "bfloat16" else _lib.F32
-        cc = _ConfigC(self.width_p, cfg.width, cfg.vocab, len(cfg.layers), batch, max_tokens, chunk, dt, cfg.eps)
+    def _create(self, chunk, dtype):
+        cfg = self.cfg
+        cc = _ConfigC(self.width_p, cfg.width, cfg.vocab, len(cfg.layers), self.batch, self.max_tokens, chunk, dtype, cfg.eps)
         lc = (_LayerC * len(cfg.layers))()
         self.head_dims = []
         for i, x in enumerate(cfg.layers):
             d, dv = self._pad_head(x.dim, x.vdim)
             self.head_dims.append((d, dv))
-            lc[i] = _LayerC(x.heads, x.kv_heads, d, dv, x.window, int(x.v_mix), x.mlp, _up8(x.ff), x.experts, x.identity,
+            lc[i] = _LayerC(x.heads, x.kv_heads, d, dv, x.window, int(x.v_mix), x.mlp, up8(x.ff), x.experts, x.identity,
                             x.top, x.groups, x.keep, x.scale, x.softcap)
         mixing = [x.kv_heads * 1000003 + x.vdim for x in cfg.layers if x.v_mix]
         if len(set(mixing)) > 1:
             raise ValueError("layers that mix values must have the same kv_heads and vdim")
-        h = self.L.ytcuda_duzozen_create(C.byref(cc), C.cast(lc, C.c_void_p))
-        if not h:
-            raise _lib.YtCudaInvalidArgument(_lib.INVALID_ARG, _lib.last_error())
-        self.h = C.c_void_p(h)
-        self._keep = []
+        return cc, lc
 
     def _pad_head(self, dim: int, vdim: int):
         if self.dtype == "bfloat16":
             for size in (64, 128):  # what the tensor-core attention takes
                 if max(dim, vdim) <= size:
                     return size, size
-        return _up8(dim), _up8(vdim)
+        return up8(dim), up8(vdim)
 
-    # ---- weights
-    def load_weights(self, weights) -> None:
-        """weights: checkpoint name -> numpy array (uint16: bf16 bits, or float32) or torch tensor; anything with
-        __getitem__ (a dict, a SafetensorsFile)."""
-        torch = self.torch
-        dev = torch.device("cuda", torch.cuda.current_device())
-        pad = torch.nn.functional.pad
-        cfg, wp = self.cfg, self.width_p
-        shapes = cfg.tensor_shapes()
-
-        def get(name, dtype):
-            a = weights[name]
-            if not isinstance(a, torch.Tensor):
-                a = np.array(a)  # (an own, writable copy)
-                a = torch.from_numpy(a.view(np.int16)).view(torch.bfloat16) if a.dtype == np.uint16 else torch.from_numpy(a)
-            if tuple(a.shape) != shapes[name]:
-                raise ValueError(f"{name}: shape {tuple(a.shape)} does not fit the configuration ({shapes[name]})")
-            return a.to(dev).to(dtype)
-
-        def mat(name, rows=0, cols=0):  # zero-padded to rows x cols (0: as it is)
-            a = get(name, torch.bfloat16)
-            return pad(a, (0, max(0, cols - a.shape[1]), 0, max(0, rows - a.shape[0])))
-
-        def vec(name, size=0):
-            a = get(name, torch.float32).reshape(-1)
-            return pad(a, (0, max(0, size - a.shape[0])))
-
-        def heads_in(name, n, d, dp):   # [n * d, width] -> [n * dp, width_p]
-            a = get(name, torch.bfloat16).reshape(n, d, cfg.width)
-            return pad(a, (0, wp - cfg.width, 0, dp - d)).reshape(n * dp, wp)
-
-        def put(name, layer, t):
-            t = t.contiguous()
-            self._keep.append(t)
-            check(self.L.ytcuda_duzozen_set_weight(self.h, name.encode(), layer, t.data_ptr()))
-
-        put("embed", 0, mat("embed", cols=wp))
-        put("head", 0, mat("head", cols=wp))
-        put("norm", 0, vec("final.norm", wp))
+    def _load(self, ck):
+        cfg, wp, put = self.cfg, self.width_p, self._put
         for i, x in enumerate(cfg.layers):
             p = f"l{i}."
             dp, dvp = self.head_dims[i]
             for n in ("norm1", "norm1b") + (("norm2", "norm2b") if x.mlp != MLP_NONE else ()):
-                put(n, i, vec(p + n, wp))
-            put("qkv", i, torch.cat([heads_in(p + "mix.q", x.heads, x.dim, dp), heads_in(p + "mix.k", x.kv_heads, x.dim, dp),
-                                     heads_in(p + "mix.v", x.kv_heads, x.vdim, dvp)]))
-            o = get(p + "mix.o", torch.bfloat16).reshape(cfg.width, x.heads, x.vdim)
-            put("o", i, pad(o, (0, dvp - x.vdim, 0, 0, 0, wp - cfg.width)).reshape(wp, x.heads * dvp))
+                put(n, i, ck.vec(p + n, wp))
+            put("qkv", i, self.torch.cat([ck.heads_out(p + "mix.q", x.heads, x.dim, dp, wp),
+                                          ck.heads_out(p + "mix.k", x.kv_heads, x.dim, dp, wp),
+                                          ck.heads_out(p + "mix.v", x.kv_heads, x.vdim, dvp, wp)]))
+            put("o", i, ck.heads_in(p + "mix.o", x.heads, x.vdim, dvp, wp))
             if x.v_mix:
-                put("vmix", i, vec(p + "mix.vmix"))
-            fp = _up8(x.ff)
+                put("vmix", i, ck.vec(p + "mix.vmix"))
+            fp = up8(x.ff)
             if x.mlp == MLP_DENSE:
-                put("up", i, mat(p + "mlp.up", fp, wp))
-                put("down", i, mat(p + "mlp.down", wp, fp))
+                put("up", i, ck.mat(p + "mlp.up", fp, wp))
+                put("down", i, ck.mat(p + "mlp.down", wp, fp))
             elif x.mlp == MLP_MOE:
-                put("router", i, mat(p + "mlp.router", cols=wp))
-                put("correction", i, vec(p + "mlp.correction"))
+                put("router", i, ck.mat(p + "mlp.router", cols=wp))
+                put("correction", i, ck.vec(p + "mlp.correction"))
                 if x.experts:
-                    gate_up = torch.zeros(x.experts, fp, 2, wp, dtype=torch.bfloat16, device=dev)
-                    down = torch.zeros(x.experts, wp, fp, dtype=torch.bfloat16, device=dev)
-                    for e in range(x.experts):
-                        q = f"{p}mlp.e{e}."
-                        gate_up[e, :, 0] = mat(q + "gate", fp, wp)
-                        gate_up[e, :, 1] = mat(q + "up", fp, wp)
-                        down[e] = mat(q + "down", wp, fp)
-                    put("up", i, gate_up)
+                    up, down = ck.experts(p + "mlp.", x.experts, fp, wp)
+                    put("up", i, up)
                     put("down", i, down)
-
-    # ---- sequences
-    def reset_kv_cache(self) -> None:
-        check(self.L.ytcuda_duzozen_reset(self.h))
-
-    def get_kv_cache_len(self) -> int:
-        return self.L.ytcuda_duzozen_cache_len(self.h)
-
-    def set_decode_path(self, path: int) -> None:
-        """One new token of a single sequence: 0 the CUDA graph of fused decode kernels, 1 one launch per operator."""
-        check(self.L.ytcuda_duzozen_set_decode_path(self.h, int(path)))
-
-    def forward_rows(self, ids, want):
-        """ids int32 [batch, len] (device) -> logits fp32 [len(want), vocab] of rows `want` of the flattened input."""
-        torch = self.torch
-        assert ids.is_cuda and ids.dtype == torch.int32 and ids.shape[0] == self.batch and ids.is_contiguous()
-        logits = torch.empty(len(want), self.cfg.vocab, dtype=torch.float32, device=ids.device)
-        rows = (C.c_int32 * len(want))(*want)
-        check(self.L.ytcuda_duzozen_forward(self.h, ids.data_ptr(), ids.shape[1], C.cast(rows, C.c_void_p), len(want),
-                                            logits.data_ptr(), torch.cuda.current_stream().cuda_stream))
-        return logits
-
-    def forward(self, ids):
-        n = ids.shape[1]
-        return self.forward_rows(ids, [b * n + n - 1 for b in range(self.batch)])
-
-    def forward_at(self, ids, want):
-        return self.forward_rows(ids, list(want))
-
-    def close(self) -> None:
-        if getattr(self, "h", None):
-            self.L.ytcuda_duzozen_destroy(self.h)
-            self.h = None
-            self._keep = []
-
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass

@@ -12,6 +12,7 @@ from typing import Callable
 
 # sources (csrc/*.cu) every model is linked with
 _CORE = ("runtime", "gemm", "flash_attn", "rowops", "sampling", "lm_rows")
+_NATIVE = _CORE + ("moe", "lm_decode", "lm_model")
 
 
 @dataclass(frozen=True)
@@ -22,12 +23,21 @@ class Model:
     load: Callable           # (folder, config dict, dtype, batch, max_tokens) -> CausalLM
 
 
-def _load_duzozen(folder: Path, config: dict, dtype: str, batch: int, max_tokens: int):
-    from .duzozen import DuzozenConfig, DuzozenForCausalLM
+def _native(config_class, model_class, folder: Path, config: dict, dtype: str, batch: int, max_tokens: int):
     from .safetensors import SafetensorsFile
-    m = DuzozenForCausalLM(DuzozenConfig.from_dict(config), batch=batch, max_tokens=max_tokens, dtype=dtype)
+    m = model_class(config_class.from_dict(config), batch=batch, max_tokens=max_tokens, dtype=dtype)
     m.load_weights(SafetensorsFile(folder / "model.safetensors"))
     return m
+
+
+def _load_duzozen(*args):
+    from .duzozen import DuzozenConfig, DuzozenForCausalLM
+    return _native(DuzozenConfig, DuzozenForCausalLM, *args)
+
+
+def _load_derupel(*args):
+    from .derupel import DerupelConfig, DerupelForCausalLM
+    return _native(DerupelConfig, DerupelForCausalLM, *args)
 
 
 def _load_qwen3(folder: Path, config: dict, dtype: str, batch: int, max_tokens: int):
@@ -42,7 +52,8 @@ def _load_qwen3(folder: Path, config: dict, dtype: str, batch: int, max_tokens: 
 
 
 MODELS = {
-    "Duzozen": Model("Duzozen", ("bfloat16", "float32"), _CORE + ("moe", "lm_decode", "duzozen"), _load_duzozen),
+    "Duzozen": Model("Duzozen", ("bfloat16", "float32"), _NATIVE + ("duzozen",), _load_duzozen),
+    "Derupel": Model("Derupel", ("bfloat16", "float32"), _NATIVE + ("latent_attn", "decayed_attn", "derupel"), _load_derupel),
     # (bf16 weights with fp32 activations: the one format it has)
     "Qwen3ForCausalLM": Model("Qwen3ForCausalLM", ("bfloat16",), _CORE + ("elementwise", "decoder"), _load_qwen3),
 }
