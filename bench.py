@@ -17,7 +17,7 @@ roofline, end-to-end (host buffers) and CPU-baseline legs:
   chain     rmsNorm + broadcast residual + row softmax + bf16 cast on [32,4096,4096] fp32   (N = 1 only)
   gemm32    fp32 GEMM 1024^3                                                                (N = 1 only)
   gemm_weak the headline GEMM with 64 matrices PER RANK                                     (N > 1 only)
-`--workload lm` (on request only): prefill and decode throughput of the Duzozen model at a few sizes, beside the Qwen3
+`--workload lm` (on request only): prefill and decode throughput of the Duzozen and Derupel models at a few sizes, beside the Qwen3
 decoder of equal size.
 Every secondary workload runs in a child process of its own (same rank environment, its own rendezvous port), so a
 failure there is recorded in its entry and cannot take the headline with it.
@@ -836,40 +836,107 @@ def _device_weights(torch, shapes, seed=4, std=0.02):
 
 
 def lm_sizes():
-    """Layers of the size of a real model: name -> (Duzozen configuration, Qwen3 configuration of equal size)."""
+    """Layers of the size of a real model: (model, name) -> (configuration, Qwen3 configuration of equal size)."""
     from ytensor_b200 import qwen3 as Q
-    from ytensor_b200.duzozen import MLP_DENSE, MLP_MOE, DuzozenConfig, DuzozenLayer
+    from ytensor_b200.derupel import DECAYED, LATENT, DerupelConfig, DerupelLayer
+    from ytensor_b200.duzozen import DuzozenConfig, DuzozenLayer
+    from ytensor_b200.native_lm import MLP_DENSE, MLP_MOE
 
-    def make(width, vocab, n, heads, kv, window, **mlp):
+    def duzozen(width, vocab, n, heads, kv, window, **mlp):
         att = dict(heads=heads, kv_heads=kv, dim=128, vdim=128, scale=128 ** -0.5, softcap=20.0, window=window, v_mix=True)
         dense = dict(mlp=MLP_DENSE, ff=mlp["dense"])
         rest = dict(mlp=MLP_MOE, **mlp["moe"]) if "moe" in mlp else dense
         return DuzozenConfig(width=width, vocab=vocab, eps=1e-6,
                              layers=[DuzozenLayer(**att, **(rest if l else dense)) for l in range(n)])
 
+    def derupel(width, vocab, n, heads, kv_rank, q_rank, **mlp):  # one layer in four attends to latents
+        decay = [1 - 2.0 ** (-2 - 8.0 * h / heads) for h in range(heads)]
+        mixers = (dict(mixer=LATENT, heads=heads, dim=64, vdim=128, rot_dim=64, rot_dims=64, kv_rank=kv_rank, q_rank=q_rank,
+                       scale=128 ** -0.5),
+                  dict(mixer=DECAYED, heads=heads, dim=128, vdim=128, decay=decay))
+        dense = dict(mlp=MLP_DENSE, ff=mlp["dense"])
+        rest = dict(mlp=MLP_MOE, **mlp["moe"]) if "moe" in mlp else dense
+        return DerupelConfig(width=width, vocab=vocab, eps=1e-6, embed_scale=width ** 0.5,
+                             layers=[DerupelLayer(**mixers[l % 4 != 3], **(rest if l else dense)) for l in range(n)])
+
     small = Q.Qwen3Config(max_position_embeddings=8192)
     large = Q.Qwen3Config(hidden_size=4096, num_hidden_layers=8, vocab_size=32768, intermediate_size=9600,
                           num_attention_heads=32, num_key_value_heads=8, max_position_embeddings=8192)
     return {
-        "width 1024, 28 layers, dense": (make(1024, 151936, 28, 16, 8, 1024, dense=4608), small),
-        "width 1024, 28 layers, 64 experts + 8 identity, top 8": (
-            make(1024, 151936, 28, 16, 8, 1024, dense=4608,
-                 moe=dict(ff=384, experts=64, identity=8, top=8, groups=8, keep=4)), small),
-        "width 4096, 8 layers, dense": (make(4096, 32768, 8, 32, 8, 2048, dense=14400), large),
-        "width 4096, 8 layers, 32 experts + 4 identity, top 4": (
-            make(4096, 32768, 8, 32, 8, 2048, dense=14400,
-                 moe=dict(ff=2400, experts=32, identity=4, top=4, groups=6, keep=3)), large),
+        ("Duzozen", "width 1024, 28 layers, dense"): (duzozen(1024, 151936, 28, 16, 8, 1024, dense=4608), small),
+        ("Duzozen", "width 1024, 28 layers, 64 experts + 8 identity, top 8"): (
+            duzozen(1024, 151936, 28, 16, 8, 1024, dense=4608,
+                    moe=dict(ff=384, experts=64, identity=8, top=8, groups=8, keep=4)), small),
+        ("Duzozen", "width 4096, 8 layers, dense"): (duzozen(4096, 32768, 8, 32, 8, 2048, dense=14400), large),
+        ("Duzozen", "width 4096, 8 layers, 32 experts + 4 identity, top 4"): (
+            duzozen(4096, 32768, 8, 32, 8, 2048, dense=14400,
+                    moe=dict(ff=2400, experts=32, identity=4, top=4, groups=6, keep=3)), large),
+        ("Derupel", "width 1024, 28 layers, dense"): (derupel(1024, 151936, 28, 16, 512, 512, dense=4608), small),
+        ("Derupel", "width 1024, 28 layers, 64 experts, top 7 + shared"): (
+            derupel(1024, 151936, 28, 16, 512, 512, dense=4608,
+                    moe=dict(ff=384, experts=64, top=7, limit=7.0, shared_ff=384, shared_limit=7.0)), small),
+        ("Derupel", "width 4096, 8 layers, dense"): (derupel(4096, 32768, 8, 32, 512, 1536, dense=14400), large),
+        ("Derupel", "width 4096, 8 layers, 32 experts, top 3 + shared"): (
+            derupel(4096, 32768, 8, 32, 512, 1536, dense=14400,
+                    moe=dict(ff=2400, experts=32, top=3, limit=7.0, shared_ff=2400, shared_limit=7.0)), large),
     }
 
 
+def lm_work(cfg) -> dict:
+    """Algorithmic work of a model: products per token (multiply-adds), extra flops of a prompt of n tokens, bytes that a
+    decode step reads besides the weights (2 bytes per product operand) behind a context."""
+    from ytensor_b200.native_lm import MLP_DENSE, MLP_MOE
+    W = cfg.width
+    per_token = 0
+    for x in cfg.layers:
+        if hasattr(x, "mixer"):
+            per_token += 2 * W * x.heads * x.vdim  # gate, output
+            if x.kv_rank:
+                per_token += W * (x.q_rank + x.kv_rank + x.rot_dim) + x.q_rank * x.heads * (x.dim + x.rot_dim)
+                per_token += x.kv_rank * x.heads * (x.dim + x.vdim)
+            else:
+                per_token += W * x.heads * (2 * x.dim + x.vdim)
+        else:
+            per_token += W * (x.heads + x.kv_heads) * (x.dim + x.vdim)
+        if x.mlp == MLP_DENSE:
+            per_token += 2 * W * x.ff
+        elif x.mlp == MLP_MOE:
+            identity = getattr(x, "identity", 0)
+            per_token += x.top * x.experts / (x.experts + identity) * 3 * W * x.ff + (x.experts + identity) * W
+            per_token += 3 * W * getattr(x, "shared_ff", 0)
+
+    def mixer_flops(n):  # causal pairs inside the window; two products of a head's state per token
+        out = 0
+        for x in cfg.layers:
+            if hasattr(x, "mixer") and not x.kv_rank:
+                out += 4 * n * x.heads * x.dim * x.vdim
+                continue
+            span = min(n, getattr(x, "window", 0) or n)
+            out += 2 * x.heads * (x.dim + getattr(x, "rot_dim", 0) + x.vdim) * (n * span - span ** 2 / 2)
+        return out
+
+    def state_bytes(ctx):
+        out = 0
+        for x in cfg.layers:
+            if hasattr(x, "mixer"):
+                out += ctx * (x.kv_rank + x.rot_dim) * 2 if x.kv_rank else 2 * 4 * x.heads * x.dim * x.vdim  # read, written
+            else:
+                out += min(ctx, x.window or ctx) * x.kv_heads * (x.dim + x.vdim) * 2
+        return out
+
+    return {"per_token": per_token, "mixer_flops": mixer_flops, "state_bytes": state_bytes, "head": W * cfg.vocab}
+
+
 def lm_arm(args) -> list | None:
-    """Prefill and decode throughput of the Duzozen model at a few sizes beside the Qwen3 decoder of equal size (random
-    weights; one GPU, one sequence). Prefill: prompts of 512 and 4096 tokens; decode: 128 single-token steps behind the
+    """Prefill and decode throughput of the Duzozen and Derupel models at a few sizes beside the Qwen3 decoder of equal size
+    (random weights; one GPU, one sequence). Prefill: prompts of 512 and 4096 tokens; decode: 128 single-token steps behind the
     4096-token prompt (the Qwen3 decoder: also behind 512). Device time by CUDA events."""
     D = Dist()
     torch = D.torch
     from ytensor_b200 import qwen3 as Q
-    from ytensor_b200.duzozen import MLP_DENSE, MLP_MOE, DuzozenForCausalLM
+    from ytensor_b200.derupel import DerupelForCausalLM
+    from ytensor_b200.duzozen import DuzozenForCausalLM
+    classes = {"Duzozen": DuzozenForCausalLM, "Derupel": DerupelForCausalLM}
     peaks = measured_peaks()
     reps = max(3, min(args.steps, 5))
 
@@ -899,13 +966,13 @@ def lm_arm(args) -> list | None:
         return out
 
     entries, qwen_done = [], {}
-    for name, (cfg, qcfg) in lm_sizes().items():
-        if args.only and args.only not in name:
+    for (arch, name), (cfg, qcfg) in lm_sizes().items():
+        if args.only and args.only not in f"{arch}: {name}":
             continue
         sampler = ClockSampler(D.local, interval_ms=1000)
         if not args.no_clock_sampling:
             sampler.start()
-        m = DuzozenForCausalLM(cfg, max_tokens=8192)
+        m = classes[arch](cfg, max_tokens=8192)
         m.load_weights(_device_weights(torch, cfg.tensor_shapes()))
         got = measure(m, cfg.vocab, (512, 4096))
         m.close()
@@ -935,25 +1002,13 @@ def lm_arm(args) -> list | None:
             del w
             torch.cuda.empty_cache()
         clocks = sampler.stop() if not args.no_clock_sampling else None
-        W = cfg.width
-        att = sum(W * (x.heads * (x.dim + x.vdim) + x.kv_heads * (x.dim + x.vdim)) for x in cfg.layers)
-        ff = sum(2 * W * x.ff if x.mlp == MLP_DENSE else
-                 x.top * x.experts / (x.experts + x.identity) * 3 * W * x.ff + (x.experts + x.identity) * W
-                 for x in cfg.layers if x.mlp in (MLP_DENSE, MLP_MOE))
-        head = W * cfg.vocab
-
-        def kv_bytes(ctx):
-            return sum(min(ctx, x.window or ctx) * x.kv_heads * (x.dim + x.vdim) * 2 for x in cfg.layers)
-
-        def att_flops(n):  # window-limited causal pairs
-            return sum(2 * x.heads * (x.dim + x.vdim) * (n * min(n, x.window) - min(n, x.window) ** 2 / 2) for x in cfg.layers)
-
-        e = {"metric": "lm_tokens_per_s", "model": "Duzozen", "size": name, "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
+        work = lm_work(cfg)
+        e = {"metric": "lm_tokens_per_s", "model": arch, "size": name, "unit": "tok/s", "n_gpus": 1, "dtype": "bf16",
              "data": "synthetic", "repetitions": reps, "clocks": clocks,
              "config": {"l2": "weights larger than L2; prompts and weights of one size run back to back"}}
         for n, (pre, dec) in got.items():
-            flops = 2 * n * (att + ff) + att_flops(n) + 2 * head
-            bts = 2 * (att + ff + head) + kv_bytes(n + 64)
+            flops = 2 * n * work["per_token"] + work["mixer_flops"](n) + 2 * work["head"]
+            bts = 2 * (work["per_token"] + work["head"]) + work["state_bytes"](n + 64)
             e[f"prompt_{n}"] = {
                 "prefill_tokens_per_s": n / (pre * 1e-3), "prefill_ms": pre, "prefill_tflops": flops / (pre * 1e-3) / 1e12,
                 "prefill_frac_of_bf16_peak": flops / (pre * 1e-3) / 1e12 / peaks["bf16_tflops"],
@@ -1035,7 +1090,7 @@ def main() -> None:
     ap.add_argument("--no-clock-sampling", action="store_true", help="decode workload: do not run nvidia-smi beside it")
     ap.add_argument("--no-e2e", action="store_true", help="skip the host-buffer leg (profiling captures only)")
     ap.add_argument("--new-tokens", type=int, default=256, help="decode workload: tokens generated per sequence")
-    ap.add_argument("--only", default="", help="lm workload: sizes whose name contains this")
+    ap.add_argument("--only", default="", help="lm workload: sizes whose \"model: name\" contains this")
     ap.add_argument("--no-closest", action="store_true", help="lm workload: leave the Qwen3 decoder out")
     ap.add_argument("--batch", type=int, default=0,
                     help="batch items per rank and step; anything but the default is a profiling case, not a bench line")
