@@ -267,7 +267,7 @@ def linear_case(L, code, act, x, w, want, cols, limit, dtype):
     check(L.ytcuda_linear_act(code, act, x.data_ptr(), x.shape[1], w.data_ptr(), y.data_ptr(), y.shape[1], x.shape[0],
                               w.shape[0], x.shape[1], cols, limit, None, 1, stream()))
     z = np.abs(f64(x)) @ np.abs(f64(w)).T  # (bounded results are small beside the sums they come from)
-    tol = max(2e-6, 1e-7 * z.max() / np.abs(want).max()) if dtype == "float32" else 5e-3
+    tol = max(2e-6 * (1 + limit), 1e-7 * z.max() / np.abs(want).max()) if dtype == "float32" else 5e-3
     assert normwise(f64(y), want) < tol, (act, cols, limit)
 
 

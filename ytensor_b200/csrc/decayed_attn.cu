@@ -124,12 +124,10 @@ constexpr int DC_TILE = 2 * DC_BOX;
 constexpr int DC_STATE = DC * DC;            // elements of a state
 
 struct DecayedChunks {
-  float* own;           // [units][DC][DC] fp32: a chunk's own contribution to the state
+  const float* own;     // [units][DC][DC] fp32: a chunk's own contribution to the state
   uint16_t* planes;     // [units][2][DC][DC] bf16: the state before the chunk, hi and lo
   const float* decay;
   float* state;         // [batch][heads][DC][DC]
-  void* o;
-  int64_t ld_o;
   int heads, chunks, len, first;
   int* status;
   // unit of (batch, head, chunk)
@@ -164,11 +162,12 @@ __device__ __forceinline__ void drain(uint64_t* bar) {
 
 // own = sum over s of k_s (w^(n-1-s) v_s)^T: K^T is the M operand (dims x tokens, unit stride along the dims), the decayed
 // values the N operand.
-constexpr int DS_THREADS = 128;
+constexpr int DS_THREADS = 256;
 constexpr int DS_SMEM = 3 * DC_TILE + 1024;
-__global__ void __launch_bounds__(DS_THREADS) decayed_chunk_state_kernel(const __grid_constant__ CUtensorMap tmK,
-                                                                         const __grid_constant__ CUtensorMap tmV,
-                                                                         const DecayedChunks p) {
+__global__ void __launch_bounds__(DS_THREADS, 2) decayed_chunk_state_kernel(const __grid_constant__ CUtensorMap tmK,
+                                                                            const __grid_constant__ CUtensorMap tmV,
+                                                                            const __grid_constant__ CUtensorMap tmU,
+                                                                            const DecayedChunks p) {
   extern __shared__ uint8_t ds_raw[];
   __shared__ uint64_t bars[2];
   __shared__ uint32_t tmem_slot;
@@ -237,15 +236,26 @@ __global__ void __launch_bounds__(DS_THREADS) decayed_chunk_state_kernel(const _
     ok = mbar_wait(&bars[1], 0, abort_word);
     tc_fence_after();
     if (__syncthreads_and(ok)) {
-      float* out = p.own + p.unit(b, h, c) * DC_STATE + (warp * 32 + lane) * DC;
-#pragma unroll 1
-      for (int c0 = 0; c0 < DC; c0 += 32) {
+      // rows of 32 floats in the store's 128-byte swizzle, over the operands that have been read
+      const int t = (warp & 3) * 32 + lane;
+#pragma unroll
+      for (int q = (warp >> 2) * 2; q < (warp >> 2) * 2 + 2; ++q) {
         uint32_t r[32];
-        tmem_ld_32x32b_x32(t_d + c0 + (static_cast<uint32_t>(warp * 32) << 16), r);
+        tmem_ld_32x32b_x32(t_d + q * 32 + (static_cast<uint32_t>((warp & 3) * 32) << 16), r);
         tmem_ld_wait();
 #pragma unroll
-        for (int e = 0; e < 32; e += 4)
-          *reinterpret_cast<uint4*>(out + c0 + e) = make_uint4(r[e], r[e + 1], r[e + 2], r[e + 3]);
+        for (int j = 0; j < 8; ++j)
+          *reinterpret_cast<uint4*>(smem + q * DC_BOX + t * 128 + ((j ^ (t & 7)) << 4)) =
+              make_uint4(r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
+      }
+      fence_proxy_async_smem();
+      __syncthreads();
+      if (threadIdx.x == 0) {
+        const int row = static_cast<int>(p.unit(b, h, c) * DC);
+#pragma unroll
+        for (int q = 0; q < 4; ++q) tma_store_2d(&tmU, smem + q * DC_BOX, q * 32, row);
+        tma_store_commit();
+        tma_store_wait_all<0>();
       }
     }
   } else if (threadIdx.x == 0) {
@@ -294,162 +304,182 @@ __global__ void __launch_bounds__(DN_THREADS) decayed_chunk_scan_kernel(const De
   *reinterpret_cast<float4*>(state) = s;
 }
 
-// Outputs of one chunk: S = Q K^T and Q times the state (hi, lo) as soon as they arrive; the decayed lower triangle of S goes
-// back to tensor memory as hi and lo; the product with V joins in the epilogue, which owns a row per thread.
-constexpr int DO_THREADS = 256;
-constexpr int DO_SMEM = 5 * DC_TILE + 1024;
-__global__ void __launch_bounds__(DO_THREADS) decayed_chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ,
-                                                                       const __grid_constant__ CUtensorMap tmK,
-                                                                       const __grid_constant__ CUtensorMap tmV,
-                                                                       const __grid_constant__ CUtensorMap tmS,
-                                                                       const DecayedChunks p) {
+// Outputs of one chunk. One warp loads and issues: S = Q K^T, then, over K's place in shared memory, the state before the
+// chunk (hi, lo) for C = Q S; eight warps turn S into the decayed lower triangle P (hi, lo) in tensor memory, over S, and
+// take C into registers; P V goes over C. Three tiles of shared memory and half of tensor memory: two CTAs per SM.
+constexpr int DO_WORKERS = 256, DO_THREADS = DO_WORKERS + 32;
+constexpr int DO_SMEM = 3 * DC_TILE + 1024;
+enum { DO_QK = 0, DO_V, DO_STATE, DO_S, DO_HI_DONE, DO_C, DO_P, DO_O, DO_BARS };
+__device__ __forceinline__ void workers_sync() { asm volatile("bar.sync 1, %0;" ::"n"(DO_WORKERS) : "memory"); }
+__global__ void __launch_bounds__(DO_THREADS, 2) decayed_chunk_out_kernel(const __grid_constant__ CUtensorMap tmQ,
+                                                                          const __grid_constant__ CUtensorMap tmK,
+                                                                          const __grid_constant__ CUtensorMap tmV,
+                                                                          const __grid_constant__ CUtensorMap tmS,
+                                                                          const __grid_constant__ CUtensorMap tmO,
+                                                                          const DecayedChunks p) {
   extern __shared__ uint8_t do_raw[];
-  __shared__ uint64_t bars[4];  // Q and K, V and the state, S ready, outputs ready
+  __shared__ uint64_t bars[DO_BARS];
   __shared__ uint32_t tmem_slot;
   __shared__ int abort_flag;
   __shared__ float pw[DC + 1];
   uint8_t* smem = do_raw + ((1024u - (smem_u32(do_raw) & 1023u)) & 1023u);
-  uint8_t *q_s = smem, *k_s = smem + DC_TILE, *v_s = smem + 2 * DC_TILE, *st_s = smem + 3 * DC_TILE;  // st_s: hi, lo
+  uint8_t *q_s = smem, *k_s = smem + DC_TILE, *v_s = smem + 2 * DC_TILE;
   volatile int* abort_word = &abort_flag;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int c = blockIdx.x, h = blockIdx.y, b = blockIdx.z;
   const bool carried = c > 0 || !p.first;  // (the state before the first chunk of a sequence is zero)
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 4; ++i) mbar_init(&bars[i], 1);
+    for (int i = 0; i < DO_BARS; ++i) mbar_init(&bars[i], i == DO_P ? DO_WORKERS / 32 : 1);
     abort_flag = 0;
     fence_mbar_init();
     fence_proxy_async_smem();
-    tma_prefetch_desc(&tmQ);
-    tma_prefetch_desc(&tmK);
-    tma_prefetch_desc(&tmV);
-    tma_prefetch_desc(&tmS);
   }
-  if (warp == 1) {
-    tmem_alloc(&tmem_slot, 512);
+  if (warp == DO_WORKERS / 32) {
+    tmem_alloc(&tmem_slot, 256);
     tmem_relinquish();
   }
   decay_powers(pw, p.decay[h]);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t t_s = tmem_slot, t_o = t_s + 128, t_c = t_s + 256, t_hi = t_s + 384, t_lo = t_s + 448;
+  const uint32_t t_s = tmem_slot, t_o = t_s + 128, t_hi = t_s, t_lo = t_s + 64;
   dependent_wait();
   dependent_trigger();
-  bool ok = true;
-  if (threadIdx.x == 0) {
-    mbar_expect_tx(&bars[0], 2 * DC_TILE);
-    load_tile(q_s, &tmQ, &bars[0], c * DC, h, b);
-    load_tile(k_s, &tmK, &bars[0], c * DC, h, b);
-    mbar_expect_tx(&bars[1], (carried ? 3 : 1) * DC_TILE);
-    load_tile(v_s, &tmV, &bars[1], c * DC, h, b);
-    if (carried) {
-      const int row = static_cast<int>(p.unit(b, h, c) * 2 * DC);
+  if (warp == DO_WORKERS / 32) {
+    if (lane == 0) {
+      mbar_expect_tx(&bars[DO_QK], 2 * DC_TILE);
+      load_tile(q_s, &tmQ, &bars[DO_QK], c * DC, h, b);
+      load_tile(k_s, &tmK, &bars[DO_QK], c * DC, h, b);
+      mbar_expect_tx(&bars[DO_V], DC_TILE);
+      load_tile(v_s, &tmV, &bars[DO_V], c * DC, h, b);
+      const uint32_t qa = smem_u32(q_s), ka = smem_u32(k_s), va = smem_u32(v_s);
+      bool ok = mbar_wait(&bars[DO_QK], 0, abort_word);
+      if (ok) {
+        const uint32_t idesc = umma_idesc(1u, 0, 0, DC, DC);
 #pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        tma_load_2d(st_s + i * DC_TILE, &tmS, &bars[1], 0, row + i * DC);
-        tma_load_2d(st_s + i * DC_TILE + DC_BOX, &tmS, &bars[1], 64, row + i * DC);
+        for (int kk = 0; kk < DC / 16; ++kk) {
+          const uint32_t off = (kk >> 2) * DC_BOX + (kk & 3) * 32;
+          tc_mma_f16(t_s, umma_smem_desc_sw128(qa + off, 16, 1024), umma_smem_desc_sw128(ka + off, 16, 1024), idesc,
+                     kk != 0 ? 1u : 0u);
+        }
+        tc_commit(&bars[DO_S]);
       }
-    }
-    ok = mbar_wait(&bars[0], 0, abort_word);
-    if (ok) {
-      const uint32_t qa = smem_u32(q_s), ka = smem_u32(k_s);
-      const uint32_t idesc = umma_idesc(1u, 0, 0, DC, DC);
-#pragma unroll
-      for (int kk = 0; kk < DC / 16; ++kk) {
-        const uint32_t off = (kk >> 2) * DC_BOX + (kk & 3) * 32;
-        tc_mma_f16(t_s, umma_smem_desc_sw128(qa + off, 16, 1024), umma_smem_desc_sw128(ka + off, 16, 1024), idesc,
-                   kk != 0 ? 1u : 0u);
-      }
-      tc_commit(&bars[2]);
-      ok = mbar_wait(&bars[1], 0, abort_word);
-      if (ok && carried) {
-        const uint32_t idesc_c = umma_idesc(1u, 0, 1, DC, DC);
-#pragma unroll
-        for (int i = 0; i < 2; ++i)
+      if (carried) {
+        const uint32_t idesc = umma_idesc(1u, 0, 1, DC, DC);
+        const int row = static_cast<int>(p.unit(b, h, c) * 2 * DC);
+#pragma unroll 1
+        for (int i = 0; i < 2 && ok; ++i) {  // (what stood in K's place has been read: S, then C's first half, are done)
+          ok = mbar_wait(&bars[i == 0 ? DO_S : DO_HI_DONE], 0, abort_word);
+          if (!ok) break;
+          mbar_expect_tx(&bars[DO_STATE], DC_TILE);
+          tma_load_2d(k_s, &tmS, &bars[DO_STATE], 0, row + i * DC);
+          tma_load_2d(k_s + DC_BOX, &tmS, &bars[DO_STATE], 64, row + i * DC);
+          ok = mbar_wait(&bars[DO_STATE], static_cast<uint32_t>(i), abort_word);
+          if (!ok) break;
 #pragma unroll
           for (int kk = 0; kk < DC / 16; ++kk) {
             const uint32_t off = (kk >> 2) * DC_BOX + (kk & 3) * 32;
-            tc_mma_f16(t_c, umma_smem_desc_sw128(qa + off, 16, 1024),
-                       umma_smem_desc_sw128(smem_u32(st_s) + i * DC_TILE + kk * 2048, DC_BOX, 1024), idesc_c,
+            tc_mma_f16(t_o, umma_smem_desc_sw128(qa + off, 16, 1024), umma_smem_desc_sw128(ka + kk * 2048, DC_BOX, 1024), idesc,
                        (i != 0 || kk != 0) ? 1u : 0u);
           }
-      }
-    }
-    if (!ok) {
-      drain(&bars[0]);
-      drain(&bars[1]);
-    }
-  }
-  __syncwarp();
-  if (ok) ok = mbar_wait(&bars[2], 0, abort_word);
-  tc_fence_after();
-  // warps 0 - 3 take the first 64 columns of their rows, warps 4 - 7 the others
-  const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
-  const int t = (warp & 3) * 32 + lane, half = warp >> 2;
-  if (__syncthreads_and(ok)) {
-#pragma unroll
-    for (int c0 = 0; c0 < 64; c0 += 32) {
-      uint32_t r[32], hi[16], lo[16];
-      const int col = half * 64 + c0;
-      tmem_ld_32x32b_x32(t_s + lanes + col, r);
-      tmem_ld_wait();
-#pragma unroll
-      for (int e = 0; e < 32; e += 2) {
-        const int d = t - (col + e);  // tokens between the key and this row
-        const float x = d >= 0 ? __uint_as_float(r[e]) * pw[d] : 0.f;
-        const float y = d >= 1 ? __uint_as_float(r[e + 1]) * pw[d - 1] : 0.f;
-        split_pair(x, y, hi[e >> 1], lo[e >> 1]);
-      }
-      tmem_st_32x32b_x16(t_hi + lanes + (col >> 1), hi);
-      tmem_st_32x32b_x16(t_lo + lanes + (col >> 1), lo);
-    }
-    tmem_st_wait();
-    tc_fence_before();
-    __syncthreads();
-    if (threadIdx.x == 0) {
-      tc_fence_after();
-      const uint32_t idesc_v = umma_idesc(1u, 0, 1, DC, DC);
-      const uint32_t va = smem_u32(v_s);
-#pragma unroll
-      for (int i = 0; i < 2; ++i)
-#pragma unroll
-        for (int kk = 0; kk < DC / 16; ++kk)
-          tc_mma_f16_ts(t_o, (i ? t_lo : t_hi) + kk * 8, umma_smem_desc_sw128(va + kk * 2048, DC_BOX, 1024), idesc_v,
-                        (i != 0 || kk != 0) ? 1u : 0u);
-      tc_commit(&bars[3]);
-    }
-    __syncwarp();
-    ok = mbar_wait(&bars[3], 0, abort_word);
-    tc_fence_after();
-    if (__syncthreads_and(ok)) {
-      const int row = c * DC + t;
-      const float f = pw[t + 1];
-      uint16_t* out = static_cast<uint16_t*>(p.o) + (static_cast<int64_t>(b) * p.len + row) * p.ld_o + h * DC;
-#pragma unroll
-      for (int c0 = 0; c0 < 64; c0 += 32) {
-        uint32_t r[32], s[32];
-        const int col = half * 64 + c0;
-        tmem_ld_32x32b_x32(t_o + lanes + col, r);
-        if (carried) tmem_ld_32x32b_x32(t_c + lanes + col, s);
-        tmem_ld_wait();
-        if (row < p.len) {
-#pragma unroll
-          for (int e = 0; e < 32; e += 8) {
-            float v[8];
-#pragma unroll
-            for (int k = 0; k < 8; ++k)
-              v[k] = carried ? fmaf(f, __uint_as_float(s[e + k]), __uint_as_float(r[e + k])) : __uint_as_float(r[e + k]);
-            Vec8<uint16_t>::store(out + col + e, v);
-          }
+          tc_commit(&bars[i == 0 ? DO_HI_DONE : DO_C]);
         }
       }
+      ok = ok && mbar_wait(&bars[DO_V], 0, abort_word) && mbar_wait(&bars[DO_P], 0, abort_word);
+      if (ok) {
+        tc_fence_after();
+        const uint32_t idesc = umma_idesc(1u, 0, 1, DC, DC);
+#pragma unroll
+        for (int i = 0; i < 2; ++i)
+#pragma unroll
+          for (int kk = 0; kk < DC / 16; ++kk)
+            tc_mma_f16_ts(t_o, (i ? t_lo : t_hi) + kk * 8, umma_smem_desc_sw128(va + kk * 2048, DC_BOX, 1024), idesc,
+                          (i != 0 || kk != 0) ? 1u : 0u);
+        tc_commit(&bars[DO_O]);
+      } else {
+        drain(&bars[DO_QK]);
+        drain(&bars[DO_V]);
+      }
     }
+    __syncwarp();
+  } else {
+    // warps 0 - 3 take the first 64 columns of their rows, warps 4 - 7 the others
+    const uint32_t lanes = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const int t = (warp & 3) * 32 + lane, half = warp >> 2;
+    bool ok = mbar_wait(&bars[DO_S], 0, abort_word);
+    tc_fence_after();
+    __syncwarp();
+    {
+      uint32_t hi[32], lo[32];
+#pragma unroll
+      for (int c0 = 0; c0 < 64; c0 += 32) {
+        uint32_t r[32];
+        const int col = half * 64 + c0;
+        tmem_ld_32x32b_x32(t_s + lanes + col, r);
+        tmem_ld_wait();
+#pragma unroll
+        for (int e = 0; e < 32; e += 2) {
+          const int d = t - (col + e);  // tokens between the key and this row
+          const float x = d >= 0 ? __uint_as_float(r[e]) * pw[d] : 0.f;
+          const float y = d >= 1 ? __uint_as_float(r[e + 1]) * pw[d - 1] : 0.f;
+          split_pair(x, y, hi[(c0 + e) >> 1], lo[(c0 + e) >> 1]);
+        }
+      }
+      tc_fence_before();
+      workers_sync();  // (both halves of the row have been read)
+      tc_fence_after();
+      tmem_st_32x32b_x32(t_hi + lanes + half * 32, hi);
+      tmem_st_32x32b_x32(t_lo + lanes + half * 32, lo);
+      tmem_st_wait();
+    }
+    uint32_t cr[2][32];
+    if (carried) {
+      ok = ok && mbar_wait(&bars[DO_C], 0, abort_word);
+      __syncwarp();
+      tc_fence_after();
+      tmem_ld_32x32b_x32(t_o + lanes + half * 64, cr[0]);
+      tmem_ld_32x32b_x32(t_o + lanes + half * 64 + 32, cr[1]);
+      tmem_ld_wait();
+    } else {
+#pragma unroll
+      for (int e = 0; e < 32; ++e) cr[0][e] = cr[1][e] = 0u;
+    }
+    tc_fence_before();
+    __syncwarp();
+    if (lane == 0 && ok) mbar_arrive(&bars[DO_P]);
+    ok = mbar_wait(&bars[DO_O], 0, abort_word);
+    __syncwarp();
+    tc_fence_after();
+    const float f = pw[t + 1];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {  // into Q's place, in the store's 128-byte swizzle
+      uint32_t r[32];
+      tmem_ld_32x32b_x32(t_o + lanes + half * 64 + i * 32, r);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; e += 8) {
+        float v[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] = fmaf(f, __uint_as_float(cr[i][e + k]), __uint_as_float(r[e + k]));
+        const int j = i * 4 + (e >> 3);
+        Vec8<uint16_t>::store(reinterpret_cast<uint16_t*>(q_s + half * DC_BOX + t * 128 + ((j ^ (t & 7)) << 4)), v);
+      }
+    }
+    fence_proxy_async_smem();
+    workers_sync();
+    if (threadIdx.x == 0 && ok && *abort_word == 0) {  // (rows behind the input's end are not stored)
+      tma_store_4d(&tmO, q_s, 0, c * DC, h, b);
+      tma_store_4d(&tmO, q_s + DC_BOX, 64, c * DC, h, b);
+      tma_store_commit();
+      tma_store_wait_all<0>();
+    }
+    __syncwarp();
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) {
+  if (warp == DO_WORKERS / 32) {
     tc_fence_after();
-    tmem_dealloc(t_s, 512);
+    tmem_dealloc(t_s, 256);
   }
   if (threadIdx.x == 0 && abort_flag) atomicExch(p.status, YTC_TIMEOUT);
 }
@@ -460,9 +490,10 @@ static bool chunks_allowed(const DecayedAttn& a) {
          aligned(a.k) && aligned(a.v) && aligned(a.o);
 }
 
-static int token_map(CUtensorMap* m, const void* base, const DecayedAttn& a, int batch) {  // {column, token, head, sequence}
+static int token_map(CUtensorMap* m, const void* base, int64_t ld, const DecayedAttn& a, int batch) {
+  // {column, token, head, sequence}
   const uint64_t dims[4] = {DC, static_cast<uint64_t>(a.len), static_cast<uint64_t>(a.heads), static_cast<uint64_t>(batch)};
-  const uint64_t strides[3] = {static_cast<uint64_t>(a.ld) * 2, DC * 2, static_cast<uint64_t>(a.ld) * a.len * 2};
+  const uint64_t strides[3] = {static_cast<uint64_t>(ld) * 2, DC * 2, static_cast<uint64_t>(ld) * a.len * 2};
   const uint32_t box[4] = {64, DC, 1, 1};
   return encode_tensor_map(m, CU_TENSOR_MAP_DATA_TYPE_UINT16, 4, base, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
 }
@@ -499,24 +530,27 @@ static int decayed_chunks(const DecayedAttn& all, cudaStream_t st) {
     p.planes = reinterpret_cast<uint16_t*>(ws + group * per_seq * DC_STATE * 4);
     p.decay = a.decay;
     p.state = a.state + b0 * static_cast<int64_t>(a.heads) * DC_STATE;
-    p.o = static_cast<char*>(a.o) + static_cast<int64_t>(b0) * a.len * a.ld_o * 2;
-    p.ld_o = a.ld_o;
+    a.o = static_cast<char*>(a.o) + static_cast<int64_t>(b0) * a.len * a.ld_o * 2;
     p.heads = a.heads; p.chunks = chunks; p.len = a.len; p.first = a.first ? 1 : 0;
     p.status = status;
-    CUtensorMap tmQ, tmK, tmV, tmS;
-    if ((s = token_map(&tmQ, a.q, a, nb)) != YTC_OK) return s;
-    if ((s = token_map(&tmK, a.k, a, nb)) != YTC_OK) return s;
-    if ((s = token_map(&tmV, a.v, a, nb)) != YTC_OK) return s;
+    CUtensorMap tmQ, tmK, tmV, tmO, tmU, tmS;
+    if ((s = token_map(&tmQ, a.q, a.ld, a, nb)) != YTC_OK) return s;
+    if ((s = token_map(&tmK, a.k, a.ld, a, nb)) != YTC_OK) return s;
+    if ((s = token_map(&tmV, a.v, a.ld, a, nb)) != YTC_OK) return s;
+    if ((s = token_map(&tmO, a.o, a.ld_o, a, nb)) != YTC_OK) return s;
     {
-      const uint64_t dims[2] = {DC, static_cast<uint64_t>(nb * per_seq * 2 * DC)}, strides[1] = {DC * 2};
-      const uint32_t box[2] = {64, DC};
-      s = encode_tensor_map(&tmS, CU_TENSOR_MAP_DATA_TYPE_UINT16, 2, p.planes, dims, strides, box, CU_TENSOR_MAP_SWIZZLE_128B);
+      const uint64_t rows = static_cast<uint64_t>(nb * per_seq) * DC;
+      const uint64_t dims_u[2] = {DC, rows}, strides_u[1] = {DC * 4}, dims_s[2] = {DC, 2 * rows}, strides_s[1] = {DC * 2};
+      const uint32_t box_u[2] = {32, DC}, box_s[2] = {64, DC};
+      s = encode_tensor_map(&tmU, CU_TENSOR_MAP_DATA_TYPE_FLOAT32, 2, p.own, dims_u, strides_u, box_u, CU_TENSOR_MAP_SWIZZLE_128B);
+      if (s != YTC_OK) return s;
+      s = encode_tensor_map(&tmS, CU_TENSOR_MAP_DATA_TYPE_UINT16, 2, p.planes, dims_s, strides_s, box_s, CU_TENSOR_MAP_SWIZZLE_128B);
       if (s != YTC_OK) return s;
     }
     const dim3 grid(chunks, a.heads, nb);
-    YTC_CUDA(launch_overlapped(decayed_chunk_state_kernel, grid, dim3(DS_THREADS), DS_SMEM, st, tmK, tmV, p));
+    YTC_CUDA(launch_overlapped(decayed_chunk_state_kernel, grid, dim3(DS_THREADS), DS_SMEM, st, tmK, tmV, tmU, p));
     YTC_CUDA(launch_overlapped(decayed_chunk_scan_kernel, dim3(DC_STATE / 4 / DN_THREADS, a.heads, nb), dim3(DN_THREADS), 0, st, p));
-    YTC_CUDA(launch_overlapped(decayed_chunk_out_kernel, grid, dim3(DO_THREADS), DO_SMEM, st, tmQ, tmK, tmV, tmS, p));
+    YTC_CUDA(launch_overlapped(decayed_chunk_out_kernel, grid, dim3(DO_THREADS), DO_SMEM, st, tmQ, tmK, tmV, tmS, tmO, p));
     count_launch(3);
     YTC_CUDA(cudaGetLastError());
   }

@@ -49,6 +49,7 @@ struct FlashParams {
   int causal_off;
   float scale_log2;          // scale * log2(e)
   int is_bf16;
+  int round_nearest;         // bf16 results rounded to nearest even in the plain form too
   int pair_heads;            // 1: the two tiles are two heads of one group; 0: two neighbouring row blocks
   int row_blocks;            // query row blocks (of one tile with head pairs, of two tiles otherwise)
   int head_slots;            // head pairs (pair_heads) or heads
@@ -833,7 +834,7 @@ __global__ void __launch_bounds__(FA_THREADS, 1)
 #pragma unroll
             for (int e = 0; e < 32; e += 2) {
               const float a0 = __uint_as_float(r[e]) * inv, a1 = __uint_as_float(r[e + 1]) * inv;
-              if (MODE != FA_PLAIN) {
+              if (MODE != FA_PLAIN || p.round_nearest) {
                 w[e >> 1] = pack_bf16x2_rn(a0, a1);
                 continue;
               }
@@ -1671,9 +1672,10 @@ static bool tc_strides_ok(const void* ptr, int64_t s_row, int64_t s_head, int64_
 
 template <int D>
 static int launch_window_tc(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const FlashParams& p,
-                            bool bounded, cudaStream_t st) {
+                            int mode, cudaStream_t st) {
   const dim3 grid(static_cast<unsigned>(p.n_items < sm_count() ? p.n_items : sm_count()));
-  auto* fn = bounded ? flash_tc_kernel<D, FA_WINDOW_BOUNDED> : flash_tc_kernel<D, FA_WINDOW>;
+  auto* fn = mode == FA_PLAIN ? flash_tc_kernel<D, FA_PLAIN>
+                              : mode == FA_WINDOW_BOUNDED ? flash_tc_kernel<D, FA_WINDOW_BOUNDED> : flash_tc_kernel<D, FA_WINDOW>;
   const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(fn), FaSmem<D>::DYN_BYTES);
   if (s != YTC_OK) return s;
   YTC_CUDA(launch_overlapped(fn, grid, dim3(FA_THREADS), FaSmem<D>::DYN_BYTES, st, tmQ, tmK, tmV, p));
@@ -1738,9 +1740,12 @@ int window_attention(const WindowAttn& a, cudaStream_t st) {
     }
     p.items_per_row_block = p.head_slots * a.batch;
     p.n_items = static_cast<int>(items);
-    const bool bounded = a.softcap > 0.f && a.softcap <= FA_BOUNDED_CAP;
-    return a.head_dim == 128 ? launch_window_tc<128>(tmQ, tmK, tmV, p, bounded, st)
-                             : launch_window_tc<64>(tmQ, tmK, tmV, p, bounded, st);
+    // (without a window key 0 is position 0 and lies in row 0: the plain kernel)
+    const int mode = a.window == 0 && a.softcap == 0.f ? FA_PLAIN
+                     : a.softcap > 0.f && a.softcap <= FA_BOUNDED_CAP ? FA_WINDOW_BOUNDED : FA_WINDOW;
+    p.round_nearest = 1;
+    return a.head_dim == 128 ? launch_window_tc<128>(tmQ, tmK, tmV, p, mode, st)
+                             : launch_window_tc<64>(tmQ, tmK, tmV, p, mode, st);
   }
   if (a.head_dim > SIMT_MAX_D || a.value_dim > SIMT_MAX_D) {
     set_last_error("window_attention: head_dim / value_dim above %d are not supported", SIMT_MAX_D);
@@ -1825,7 +1830,7 @@ int ytcuda_flash_attn_fwd(int dtype, const void* Q, const void* K, const void* V
     p.batch = batch; p.kv_heads = kv_heads; p.groups = groups; p.q_len = q_len; p.kv_len = kv_len;
     p.causal = causal; p.causal_off = causal_offset;
     p.scale_log2 = scale * FA_LOG2E;
-    p.window = p.key_tile0 = p.ring_tiles = 0;
+    p.window = p.key_tile0 = p.ring_tiles = p.round_nearest = 0;
     p.cap_log2 = p.cap_raw = p.cap_in = 0.f;
     p.is_bf16 = dtype == YTC_BF16;
     p.pair_heads = (groups % 2 == 0) ? 1 : 0;

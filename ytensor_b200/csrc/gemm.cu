@@ -172,6 +172,8 @@ __device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const u
     return;
   }
   uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + gn0;
+  // EPI_SILU: these 32 columns are all activated, none, or some
+  const bool silu = p.epi == EPI_SILU && gn0 + 32 <= p.act_cols, mixed = p.epi == EPI_SILU && !silu && gn0 < p.act_cols;
   uint32_t w[16];
 #pragma unroll
   for (int j = 0; j < 16; ++j) {
@@ -182,7 +184,10 @@ __device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const u
     } else if (p.epi == EPI_RELU2) {
       a = lm_relu2(a);
       b = lm_relu2(b);
-    } else if (p.epi == EPI_SILU) {
+    } else if (silu) {
+      a = lm_silu_fast(a);
+      b = lm_silu_fast(b);
+    } else if (mixed) {
       if (gn0 + 2 * j < p.act_cols) a = lm_silu_fast(a);
       if (gn0 + 2 * j + 1 < p.act_cols) b = lm_silu_fast(b);
     }

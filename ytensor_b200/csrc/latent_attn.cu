@@ -15,17 +15,22 @@ constexpr int LA_THREADS = 256, LA_WARPS = LA_THREADS / 32;
 constexpr int LA_HEADS = 16;       // heads that share a pass over the cache
 constexpr int LA_TILE = 64;        // cache rows per step of the tensor-core kernel
 constexpr int LA_TILE_SIMT = 32;   // of the FFMA kernel
-constexpr int LA_MAX_SPLITS = 32;
+constexpr int LA_MAX_SPLITS = 64;
 
-__device__ __forceinline__ float la_block_sum(float v, float* red) {
+// Both sums over the block, in every thread.
+__device__ __forceinline__ void la_block_sum2(float& a, float& b, float2* red) {
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  for (int o = 16; o > 0; o >>= 1) {
+    a += __shfl_xor_sync(0xffffffffu, a, o);
+    b += __shfl_xor_sync(0xffffffffu, b, o);
+  }
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
   __syncthreads();
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
-  __syncthreads();
-  float t = 0.f;
-  for (int i = 0; i < static_cast<int>(blockDim.x) / 32; ++i) t += red[i];
-  return t;
+  a = b = 0.f;
+  for (int i = 0; i < static_cast<int>(blockDim.x) / 32; ++i) {
+    a += red[i].x;
+    b += red[i].y;
+  }
 }
 template <typename T>
 __device__ __forceinline__ float la_load(const void* p, int64_t i) {
@@ -50,30 +55,40 @@ __device__ __forceinline__ void la_cp_wait() {
 // ---------------------------------------------------------------- cache append
 // One row by a whole CTA. TI: the projection's format, TC: the cache's.
 template <typename TI, typename TC>
-__device__ __forceinline__ void append_row(const LatentAppend& p, int row, float* red) {
+__device__ __forceinline__ void append_row(const LatentAppend& p, int row, float2* red) {
   const int b = row / p.len, t = row - b * p.len;
   const int64_t pos = p.pos ? *p.pos : p.pos0 + t;
   const int64_t in0 = static_cast<int64_t>(row) * p.ld;
-  if (p.cq) {
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x) {
-      const float v = la_load<TI>(p.in, in0 + p.dq_off + i);
-      ss = fmaf(v, v, ss);
-    }
-    const float inv = 1.0f / sqrtf(la_block_sum(ss, red) / p.q_width + p.eps);
-    for (int i = threadIdx.x; i < p.q_rank; i += blockDim.x)
-      la_store<TI>(p.cq, static_cast<int64_t>(row) * p.q_rank + i, la_load<TI>(p.in, in0 + p.dq_off + i) * inv * p.w_q[i]);
-  }
   const int64_t out = (static_cast<int64_t>(b) * p.cap + pos) * p.s.row();
   const int64_t c0 = in0 + p.dkv_off, r0 = c0 + p.s.rank;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < p.s.rank; i += blockDim.x) {
-    const float v = la_load<TI>(p.in, c0 + i);
-    ss = fmaf(v, v, ss);
+  // the query latent (unless the caller norms it) and the latent, side by side: pieces of 8 channels
+  const TI* in = static_cast<const TI*>(p.in);
+  const int q_pieces = p.cq ? p.q_rank / 8 : 0, pieces = q_pieces + p.s.rank / 8;
+  float sq = 0.f, sc = 0.f;
+  for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+    const bool is_q = i < q_pieces;
+    float v[8];
+    Vec8<TI>::load(in + (is_q ? in0 + p.dq_off + i * 8 : c0 + (i - q_pieces) * 8), v);
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) ss = fmaf(v[e], v[e], ss);
+    sq += is_q ? ss : 0.f;
+    sc += is_q ? 0.f : ss;
   }
-  const float inv = 1.0f / sqrtf(la_block_sum(ss, red) / p.c_width + p.eps);
-  for (int i = threadIdx.x; i < p.s.rank; i += blockDim.x)
-    la_store<TC>(p.cache, out + i, la_load<TI>(p.in, c0 + i) * inv * p.w_c[i]);
+  la_block_sum2(sq, sc, red);
+  const float inv_q = p.cq ? 1.0f / sqrtf(sq / p.q_width + p.eps) : 0.f, inv_c = 1.0f / sqrtf(sc / p.c_width + p.eps);
+  for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+    const bool is_q = i < q_pieces;
+    const int e0 = (is_q ? i : i - q_pieces) * 8;
+    float v[8], w[8];
+    Vec8<TI>::load(in + (is_q ? in0 + p.dq_off : c0) + e0, v);
+    Vec8<float>::load((is_q ? p.w_q : p.w_c) + e0, w);
+    const float inv = is_q ? inv_q : inv_c;
+#pragma unroll
+    for (int e = 0; e < 8; ++e) v[e] *= inv * w[e];
+    if (is_q) Vec8<TI>::store(static_cast<TI*>(p.cq) + static_cast<int64_t>(row) * p.q_rank + e0, v);
+    else Vec8<TC>::store(static_cast<TC*>(p.cache) + out + e0, v);
+  }
   for (int i = threadIdx.x; i < p.s.rot / 2; i += blockDim.x) {
     float u = la_load<TI>(p.in, r0 + 2 * i), v = la_load<TI>(p.in, r0 + 2 * i + 1);
     if (2 * i < p.s.rot_dims) {
@@ -90,7 +105,7 @@ __device__ __forceinline__ void append_row(const LatentAppend& p, int row, float
 
 template <typename T>
 __global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppend p) {
-  __shared__ float red[4];
+  __shared__ float2 red[4];
   dependent_wait();
   dependent_trigger();
   append_row<T, T>(p, blockIdx.x, red);
@@ -163,7 +178,7 @@ __global__ void __launch_bounds__(LA_THREADS) latent_absorb_kernel(const LatentD
                                                                    int slices) {
   __shared__ float part[LA_WARPS][128];
   __shared__ float q_s[512];
-  __shared__ float red[LA_WARPS];
+  __shared__ float2 red[LA_WARPS];
   const LatentShape& s = p.s;
   const int row = blockIdx.y;
   if (static_cast<int>(blockIdx.x) == s.heads * slices) {
@@ -301,14 +316,15 @@ __global__ void __launch_bounds__(LA_THREADS) latent_slice_mma_kernel(const Late
   slice_of(n, LA_TILE, p.splits, split, begin, end, used);
   const uint16_t* cache = static_cast<const uint16_t*>(p.cache) + (row / p.len) * p.cap * p.row;
   const int pieces = p.row / 8;
-  // rows [first, last) of the tile at key0; what lies past `last` is zero
+  // the rows of the tile at key0 before `last`, one row per warp and trip; what lies past `last` is zero
   auto fetch = [&](int64_t key0, int buf, int64_t last) {
     uint16_t* dst = kv + buf * LA_TILE * ld;
-    for (int i = threadIdx.x; i < LA_TILE * pieces; i += LA_THREADS) {
-      const int r = i / pieces, c = (i - r * pieces) * 8;
-      if (key0 + r < last) la_cp16(dst + r * ld + c, cache + (key0 + r) * p.row + c);
-      else *reinterpret_cast<uint4*>(dst + r * ld + c) = make_uint4(0u, 0u, 0u, 0u);
-    }
+#pragma unroll 4
+    for (int r = warp; r < LA_TILE; r += LA_WARPS)
+      for (int c = lane; c < pieces; c += 32) {
+        if (key0 + r < last) la_cp16(dst + r * ld + c * 8, cache + (key0 + r) * p.row + c * 8);
+        else *reinterpret_cast<uint4*>(dst + r * ld + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+      }
   };
   const int tiles = begin < end ? static_cast<int>((end - begin + LA_TILE - 1) / LA_TILE) : 0;
   // (the newest row may be written by the kernel before this one)
@@ -321,13 +337,16 @@ __global__ void __launch_bounds__(LA_THREADS) latent_slice_mma_kernel(const Late
   dependent_trigger();
   if (tiles == 0) return;
   const float* qa = p.qa + (static_cast<int64_t>(row) * p.heads + h0) * p.row;
-  for (int i = threadIdx.x; i < LA_HEADS * p.row; i += LA_THREADS) {
-    const int h = i / p.row, c = i - h * p.row;
-    uint16_t hi = 0, lo = 0;
-    if (h < nh) split_bf16(qa[i], hi, lo);
-    q_hi[h * ld + c] = hi;
-    q_lo[h * ld + c] = lo;
-  }
+  for (int h = warp; h < LA_HEADS; h += LA_WARPS)
+#pragma unroll 5
+    for (int c = lane * 4; c < p.row; c += 128) {
+      const float4 v = h < nh ? *reinterpret_cast<const float4*>(qa + h * p.row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      const uint2 hi = make_uint2(pack_bf16x2_rn(v.x, v.y), pack_bf16x2_rn(v.z, v.w));
+      *reinterpret_cast<uint2*>(q_hi + h * ld + c) = hi;
+      *reinterpret_cast<uint2*>(q_lo + h * ld + c) =
+          make_uint2(pack_bf16x2_rn(v.x - __uint_as_float(hi.x << 16), v.y - __uint_as_float(hi.x & 0xFFFF0000u)),
+                     pack_bf16x2_rn(v.z - __uint_as_float(hi.y << 16), v.w - __uint_as_float(hi.y & 0xFFFF0000u)));
+    }
   if (threadIdx.x < LA_HEADS) {
     m_s[threadIdx.x] = -CUDART_INF_F;
     l_s[threadIdx.x] = 0.f;
@@ -532,7 +551,7 @@ constexpr int LA_VROWS = 16;
 template <typename TO>
 __global__ void __launch_bounds__(LA_THREADS) latent_values_kernel(const LatentDecode p, int splits, int rows_per, int slices) {
   extern __shared__ __align__(16) uint8_t la_smem[];
-  float* ctx = reinterpret_cast<float*>(la_smem);  // [rank]
+  float* ctx = reinterpret_cast<float*>(la_smem);  // [ways][rank]
   __shared__ float w_s[LA_MAX_SPLITS];
   const LatentShape& s = p.s;
   const int row = blockIdx.y, h = blockIdx.x / slices, r0 = (blockIdx.x - h * slices) * rows_per;
@@ -556,25 +575,53 @@ __global__ void __launch_bounds__(LA_THREADS) latent_values_kernel(const LatentD
   slice_of(pos + 1, LA_TILE, splits, 0, begin, end, used);
   const int stride = s.rank + 2;
   const float* part = p.part + (static_cast<int64_t>(row) * s.heads + h) * splits * stride;
+  // four channels per thread; threads left over split the slices among them
+  const int quads = s.rank / 4, ways = quads < LA_THREADS ? LA_THREADS / quads : 1;
   if (warp == 0) {
-    const float m = lane < used ? part[lane * stride + s.rank] : -CUDART_INF_F;
-    float mx = m;
+    float m[2], l[2], mx = -CUDART_INF_F;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int k = lane + 32 * i;
+      m[i] = k < used ? part[k * stride + s.rank] : -CUDART_INF_F;
+      l[i] = k < used ? part[k * stride + s.rank + 1] : 0.f;
+      mx = fmaxf(mx, m[i]);
+    }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-    const float f = lane < used ? expf(m - mx) : 0.f;
-    float l = lane < used ? f * part[lane * stride + s.rank + 1] : 0.f;
+    float sum = 0.f;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-    w_s[lane] = f / l;
+    for (int i = 0; i < 2; ++i) {
+      m[i] = expf(m[i] - mx);
+      sum = fmaf(m[i], l[i], sum);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+#pragma unroll
+    for (int i = 0; i < 2; ++i) w_s[lane + 32 * i] = m[i] / sum;
   }
   __syncthreads();
-  for (int c = threadIdx.x; c < s.rank; c += LA_THREADS) {
-    float v = 0.f;
+  for (int q0 = 0; q0 < quads; q0 += LA_THREADS) {
+    const int q = q0 + static_cast<int>(threadIdx.x) % (quads < LA_THREADS ? quads : LA_THREADS), way = quads < LA_THREADS ? threadIdx.x / quads : 0;
+    if (q >= quads || way >= ways) continue;
+    float2 a = make_float2(0.f, 0.f), b = make_float2(0.f, 0.f);
 #pragma unroll 8
-    for (int k = 0; k < used; ++k) v = fmaf(w_s[k], part[k * stride + c], v);
-    ctx[c] = v;
+    for (int k = way; k < used; k += ways) {
+      const float w = w_s[k];
+      const float2 u = *reinterpret_cast<const float2*>(part + k * stride + q * 4), v = *reinterpret_cast<const float2*>(part + k * stride + q * 4 + 2);
+      a.x = fmaf(w, u.x, a.x); a.y = fmaf(w, u.y, a.y);
+      b.x = fmaf(w, v.x, b.x); b.y = fmaf(w, v.y, b.y);
+    }
+    *reinterpret_cast<float4*>(ctx + way * s.rank + q * 4) = make_float4(a.x, a.y, b.x, b.y);
   }
   __syncthreads();
+  if (ways > 1) {
+    for (int c = threadIdx.x; c < s.rank; c += LA_THREADS) {
+      float v = ctx[c];
+      for (int k = 1; k < ways; ++k) v += ctx[k * s.rank + c];
+      ctx[c] = v;
+    }
+    __syncthreads();
+  }
 #pragma unroll
   for (int i = 0; i < LA_VROWS / LA_WARPS; ++i) {
     const int r = warp + i * LA_WARPS;
@@ -661,7 +708,7 @@ int latent_decode(const LatentDecode& a, cudaStream_t st) {
   while (rows_per > LA_WARPS && static_cast<int64_t>(s.heads) * ((s.vdim + rows_per - 1) / rows_per) * rows < sms / 2) rows_per /= 2;
   const int slices = (s.vdim + rows_per - 1) / rows_per;
   YTC_CUDA(launch_overlapped(q16 ? latent_values_kernel<uint16_t> : latent_values_kernel<float>, dim3(s.heads * slices, rows),
-                             dim3(LA_THREADS), s.rank * sizeof(float), st, a, splits, rows_per, slices));
+                             dim3(LA_THREADS), std::max(s.rank, 4 * LA_THREADS) * sizeof(float), st, a, splits, rows_per, slices));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
