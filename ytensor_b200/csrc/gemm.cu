@@ -43,6 +43,7 @@ struct GemmTcParams {
   const uint8_t* tile_live;
   // linear layers of the language models (LinearEpilogue, lm_ops.cuh)
   int epi;                 // EPI_NONE: the store rules above; otherwise tc_store_epilogue
+  int staged;              // linear layers with 16-byte aligned rows: stores go through tc_store_staged
   int act_cols;            // EPI_SILU
   float limit, alpha_gate, shift;  // EPI_CLAMP_PAIRS
   // grouped product: every 128-row block of A belongs to one group (expert) or to none (-1, passed over); group g
@@ -51,12 +52,14 @@ struct GemmTcParams {
   int group_rows;
 };
 
+constexpr int TC_OUT_BYTES = 32 * 128;  // staging area of an epilogue warp
 template <int BN>
 struct TcSmem {
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;
   static constexpr int B_BYTES = BN * TC_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int BAR_OFFSET = TC_STAGES * STAGE_BYTES;
+  static constexpr int OUT_OFFSET = TC_STAGES * STAGE_BYTES;  // staged stores: 4 warps x 32 rows x 128 bytes
+  static constexpr int BAR_OFFSET = OUT_OFFSET + 4 * TC_OUT_BYTES;
   // full[STAGES], empty[STAGES], tmem_full[2], tmem_empty[2], tmem base word, abort word
   static constexpr int TOTAL = BAR_OFFSET + (2 * TC_STAGES + 4) * 8 + 16;
   static constexpr int DYN_BYTES = TOTAL + 1024;  // slack to align the ring to 1024 B
@@ -141,67 +144,101 @@ __device__ __forceinline__ float tc_clamped_gate(const GemmTcParams& p, float ga
   const float g = fminf(gate, p.limit), u = fminf(fmaxf(up, -p.limit), p.limit);
   return __fdividef(g, 1.f + __expf(-p.alpha_gate * g)) * (u + p.shift);
 }
-// Store with a fused activation and round-to-nearest-even narrowing (see LinearEpilogue). One thread holds 32
-// consecutive columns of one row; the gated pairs make 16 results of them.
+// The fused activation and round-to-nearest-even narrowing of 32 consecutive columns of one row (see LinearEpilogue): 16
+// words of two bf16 each, 8 for the gated pairs. One loop per activation, so that its 32 results are independent work.
+__device__ __forceinline__ void tc_activate(const GemmTcParams& p, const uint32_t (&r)[32], int gn0, uint32_t (&w)[16]) {
+  auto at = [&](int i) { return __uint_as_float(r[i]); };
+  if (p.epi == EPI_SWIGLU_PAIRS) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      w[j] = pack_bf16x2_rn(lm_silu_fast(at(4 * j)) * at(4 * j + 1), lm_silu_fast(at(4 * j + 2)) * at(4 * j + 3));
+  } else if (p.epi == EPI_CLAMP_PAIRS) {
+#pragma unroll
+    for (int j = 0; j < 8; ++j)
+      w[j] = pack_bf16x2_rn(tc_clamped_gate(p, at(4 * j), at(4 * j + 1)), tc_clamped_gate(p, at(4 * j + 2), at(4 * j + 3)));
+  } else if (p.epi == EPI_GELU_ERF) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) w[j] = pack_bf16x2_rn(lm_gelu_erf(at(2 * j)), lm_gelu_erf(at(2 * j + 1)));
+  } else if (p.epi == EPI_RELU2) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) w[j] = pack_bf16x2_rn(lm_relu2(at(2 * j)), lm_relu2(at(2 * j + 1)));
+  } else if (p.epi == EPI_SILU && gn0 + 32 <= p.act_cols) {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) w[j] = pack_bf16x2_rn(lm_silu_fast(at(2 * j)), lm_silu_fast(at(2 * j + 1)));
+  } else {
+    const int n = p.epi == EPI_SILU ? p.act_cols - gn0 : 0;  // (activated columns among these)
+#pragma unroll
+    for (int j = 0; j < 16; ++j)
+      w[j] = pack_bf16x2_rn(2 * j < n ? lm_silu_fast(at(2 * j)) : at(2 * j),
+                            2 * j + 1 < n ? lm_silu_fast(at(2 * j + 1)) : at(2 * j + 1));
+  }
+}
+__device__ __forceinline__ bool tc_pairs(const GemmTcParams& p) { return p.epi == EPI_SWIGLU_PAIRS || p.epi == EPI_CLAMP_PAIRS; }
+
+// Direct store: one thread holds 32 consecutive columns of one row; the gated pairs make 16 results of them.
 __device__ __forceinline__ void tc_store_epilogue(const GemmTcParams& p, const uint32_t (&r)[32], int64_t row_off, int gn0,
                                                   bool row_ok) {
   if (!row_ok) return;
-  if (p.epi == EPI_SWIGLU_PAIRS || p.epi == EPI_CLAMP_PAIRS) {
-    uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + (gn0 >> 1);
-    uint32_t w[8];
-#pragma unroll
-    for (int j = 0; j < 8; ++j) {
-      float a, b;
-      if (p.epi == EPI_SWIGLU_PAIRS) {
-        a = lm_silu_fast(__uint_as_float(r[4 * j])) * __uint_as_float(r[4 * j + 1]);
-        b = lm_silu_fast(__uint_as_float(r[4 * j + 2])) * __uint_as_float(r[4 * j + 3]);
-      } else {
-        a = tc_clamped_gate(p, __uint_as_float(r[4 * j]), __uint_as_float(r[4 * j + 1]));
-        b = tc_clamped_gate(p, __uint_as_float(r[4 * j + 2]), __uint_as_float(r[4 * j + 3]));
-      }
-      w[j] = pack_bf16x2_rn(a, b);
-    }
-    if (gn0 + 32 <= p.N && (reinterpret_cast<uint64_t>(dst) & 15u) == 0) {
-      reinterpret_cast<uint4*>(dst)[0] = make_uint4(w[0], w[1], w[2], w[3]);
-      reinterpret_cast<uint4*>(dst)[1] = make_uint4(w[4], w[5], w[6], w[7]);
-    } else {
-#pragma unroll
-      for (int j = 0; j < 16; ++j)
-        if (gn0 + 2 * j + 1 < p.N) dst[j] = static_cast<uint16_t>(w[j >> 1] >> ((j & 1) * 16));
-    }
-    return;
-  }
-  uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + gn0;
-  // EPI_SILU: these 32 columns are all activated, none, or some
-  const bool silu = p.epi == EPI_SILU && gn0 + 32 <= p.act_cols, mixed = p.epi == EPI_SILU && !silu && gn0 < p.act_cols;
   uint32_t w[16];
+  tc_activate(p, r, gn0, w);
+  const bool pairs = tc_pairs(p);
+  uint16_t* dst = static_cast<uint16_t*>(p.C) + row_off + (pairs ? gn0 >> 1 : gn0);
 #pragma unroll
-  for (int j = 0; j < 16; ++j) {
-    float a = __uint_as_float(r[2 * j]), b = __uint_as_float(r[2 * j + 1]);
-    if (p.epi == EPI_GELU_ERF) {
-      a = lm_gelu_erf(a);
-      b = lm_gelu_erf(b);
-    } else if (p.epi == EPI_RELU2) {
-      a = lm_relu2(a);
-      b = lm_relu2(b);
-    } else if (silu) {
-      a = lm_silu_fast(a);
-      b = lm_silu_fast(b);
-    } else if (mixed) {
-      if (gn0 + 2 * j < p.act_cols) a = lm_silu_fast(a);
-      if (gn0 + 2 * j + 1 < p.act_cols) b = lm_silu_fast(b);
-    }
-    w[j] = pack_bf16x2_rn(a, b);
-  }
-  if (gn0 + 32 <= p.N && (reinterpret_cast<uint64_t>(dst) & 15u) == 0) {
+  for (int j = 0; j < 32; ++j)
+    if (j < (pairs ? 16 : 32) && (pairs ? gn0 + 2 * j + 1 : gn0 + j) < p.N)
+      dst[j] = static_cast<uint16_t>(w[j >> 1] >> ((j & 1) * 16));
+}
+
+// Store of a warp's 32 rows x 32 columns through its staging area, where a row's results gather until they fill 128 bytes;
+// then eight lanes write one row's 128 bytes (direct stores of 64 bytes per lane, a row apart, keep the epilogue behind the
+// products when k is short). buf: 32 rows of 128 bytes, 16-byte pieces exchanged by row against bank conflicts. base:
+// elements before the warp's first row, rows: how many of the 32 exist, tile_end: the tile's last column + 1.
+__device__ __forceinline__ void tc_store_staged(const GemmTcParams& p, const uint32_t (&r)[32], uint8_t* buf, int64_t base,
+                                                int rows, int gn0, int tile_end, int lane) {
+  const bool wide = p.epi == EPI_NONE, pairs = tc_pairs(p);  // (EPI_NONE: fp32 results)
+  const int esz = wide ? 4 : 2;
+  const int at = wide ? gn0 * 4 : pairs ? gn0 : gn0 * 2, bytes = wide ? 128 : pairs ? 32 : 64;  // within the output row
+  uint8_t* mine = buf + lane * 128;
+  const int piece0 = (at & 127) >> 4;
+  auto put = [&](int piece, uint32_t a, uint32_t b, uint32_t c, uint32_t d) {
+    *reinterpret_cast<uint4*>(mine + (((piece0 + piece) ^ (lane & 7)) << 4)) = make_uint4(a, b, c, d);
+  };
+  if (wide) {
 #pragma unroll
-    for (int j = 0; j < 4; ++j)
-      reinterpret_cast<uint4*>(dst)[j] = make_uint4(w[4 * j], w[4 * j + 1], w[4 * j + 2], w[4 * j + 3]);
+    for (int j = 0; j < 8; ++j) put(j, r[4 * j], r[4 * j + 1], r[4 * j + 2], r[4 * j + 3]);
   } else {
-#pragma unroll
-    for (int j = 0; j < 32; ++j)
-      if (gn0 + j < p.N) dst[j] = static_cast<uint16_t>(w[j >> 1] >> ((j & 1) * 16));
+    uint32_t w[16];
+    tc_activate(p, r, gn0, w);
+    put(0, w[0], w[1], w[2], w[3]);
+    put(1, w[4], w[5], w[6], w[7]);
+    if (!pairs) {
+      put(2, w[8], w[9], w[10], w[11]);
+      put(3, w[12], w[13], w[14], w[15]);
+    }
   }
+  if (((at + bytes) & 127) != 0 && gn0 + 32 < p.N && gn0 + 32 < tile_end) return;
+  __syncwarp();
+  const int seg = at & ~127, valid = at + bytes - seg;
+  const int row_bytes = (pairs ? p.N / 2 : p.N) * esz;
+  const int piece = lane & 7, to = seg + piece * 16;
+  char* out = static_cast<char*>(p.C) + base * esz + to;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    const int row = i * 4 + (lane >> 3);
+    const uint4 v = *reinterpret_cast<const uint4*>(buf + row * 128 + ((piece ^ (row & 7)) << 4));
+    if (row >= rows || piece * 16 >= valid || to >= row_bytes) continue;
+    char* dst = out + static_cast<int64_t>(row) * p.rsc * esz;
+    if (to + 16 <= row_bytes) {
+      *reinterpret_cast<uint4*>(dst) = v;
+    } else {
+      const uint32_t words[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int k = 0; k < 8; ++k)
+        if (to + 2 * k < row_bytes)
+          reinterpret_cast<uint16_t*>(dst)[k] = static_cast<uint16_t>(words[k >> 1] >> ((k & 1) * 16));
+    }
+  }
+  __syncwarp();
 }
 
 template <int BN>
@@ -434,7 +471,10 @@ __global__ void __launch_bounds__(TC_THREADS, 1)
         tmem_ld_wait();
         const int gn0 = nb * BN + c0;
         if (gn0 < p.N) {
-          if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
+          if (p.staged)
+            tc_store_staged(p, r, smem + S::OUT_OFFSET + q * TC_OUT_BYTES, row_off - static_cast<int64_t>(lane) * p.rsc,
+                            p.M - (gm - lane), gn0, (nb + 1) * BN, lane);
+          else if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
           else if (p.out_dtype == YTC_BF16) tc_store_chunk<BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
           else if (p.out_dtype == YTC_F32) tc_store_chunk<BN, YTC_F32>(p, r, row_off, gn0, row_ok, vec_ok);
           else tc_store_chunk<BN, YTC_F16>(p, r, row_off, gn0, row_ok, vec_ok);
@@ -471,7 +511,8 @@ struct Tc2Smem {
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;         // 128 rows of A
   static constexpr int B_BYTES = (TC2_BN / 2) * TC_BK * 2;  // 128 columns of B
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int BAR_OFFSET = TC2_STAGES * STAGE_BYTES;
+  static constexpr int OUT_OFFSET = TC2_STAGES * STAGE_BYTES;
+  static constexpr int BAR_OFFSET = OUT_OFFSET + 4 * TC_OUT_BYTES;
   static constexpr int TOTAL = BAR_OFFSET + (2 * TC2_STAGES + 4) * 8 + 16;
   static constexpr int DYN_BYTES = TOTAL + 1024;
 };
@@ -640,7 +681,10 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
         tmem_ld_wait();
         const int gn0 = nb * TC2_BN + c0;
         if (gn0 < p.N) {
-          if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
+          if (p.staged)
+            tc_store_staged(p, r, smem + S::OUT_OFFSET + q * TC_OUT_BYTES, row_off - static_cast<int64_t>(lane) * p.rsc,
+                            p.M - (gm - lane), gn0, (nb + 1) * TC2_BN, lane);
+          else if (p.epi != EPI_NONE) tc_store_epilogue(p, r, row_off, gn0, row_ok);
           else if (p.out_dtype == YTC_BF16) tc_store_chunk<TC2_BN, YTC_BF16>(p, r, row_off, gn0, row_ok, vec_ok);
           else if (p.out_dtype == YTC_F32) tc_store_chunk<TC2_BN, YTC_F32>(p, r, row_off, gn0, row_ok, vec_ok);
           else tc_store_chunk<TC2_BN, YTC_F16>(p, r, row_off, gn0, row_ok, vec_ok);
@@ -941,6 +985,8 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
   p.tile_live = nullptr;
   const LinearEpilogue none, *e = ex ? ex : &none;
   p.epi = e->epi;
+  p.staged = ex && csc == 1 && (reinterpret_cast<uint64_t>(C) & 15u) == 0 && (rsc * dtype_size(dtype_out)) % 16 == 0 &&
+             batch == 1 && (e->epi != EPI_NONE || dtype_out == YTC_F32);
   p.act_cols = e->act_cols;
   p.limit = e->limit; p.alpha_gate = e->alpha; p.shift = e->shift;
   p.tile_group = grouped ? ex->tile_group : nullptr;
