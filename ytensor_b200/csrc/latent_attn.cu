@@ -17,21 +17,6 @@ constexpr int LA_TILE = 64;        // cache rows per step of the tensor-core ker
 constexpr int LA_TILE_SIMT = 32;   // of the FFMA kernel
 constexpr int LA_MAX_SPLITS = 64;
 
-// Both sums over the block, in every thread.
-__device__ __forceinline__ void la_block_sum2(float& a, float& b, float2* red) {
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) {
-    a += __shfl_xor_sync(0xffffffffu, a, o);
-    b += __shfl_xor_sync(0xffffffffu, b, o);
-  }
-  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = make_float2(a, b);
-  __syncthreads();
-  a = b = 0.f;
-  for (int i = 0; i < static_cast<int>(blockDim.x) / 32; ++i) {
-    a += red[i].x;
-    b += red[i].y;
-  }
-}
 template <typename T>
 __device__ __forceinline__ float la_load(const void* p, int64_t i) {
   return sizeof(T) == 4 ? static_cast<const float*>(p)[i] : bf16_bits_to_f32(static_cast<const uint16_t*>(p)[i]);
@@ -53,9 +38,10 @@ __device__ __forceinline__ void la_cp_wait() {
 }
 
 // ---------------------------------------------------------------- cache append
-// One row by a whole CTA. TI: the projection's format, TC: the cache's.
+// One row by one warp. TI: the projection's format, TC: the cache's.
 template <typename TI, typename TC>
-__device__ __forceinline__ void append_row(const LatentAppend& p, int row, float2* red) {
+__device__ __forceinline__ void append_row(const LatentAppend& p, int row) {
+  const int lane = threadIdx.x & 31;
   const int b = row / p.len, t = row - b * p.len;
   const int64_t pos = p.pos ? *p.pos : p.pos0 + t;
   const int64_t in0 = static_cast<int64_t>(row) * p.ld;
@@ -65,7 +51,8 @@ __device__ __forceinline__ void append_row(const LatentAppend& p, int row, float
   const TI* in = static_cast<const TI*>(p.in);
   const int q_pieces = p.cq ? p.q_rank / 8 : 0, pieces = q_pieces + p.s.rank / 8;
   float sq = 0.f, sc = 0.f;
-  for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+#pragma unroll 4
+  for (int i = lane; i < pieces; i += 32) {
     const bool is_q = i < q_pieces;
     float v[8];
     Vec8<TI>::load(in + (is_q ? in0 + p.dq_off + i * 8 : c0 + (i - q_pieces) * 8), v);
@@ -75,9 +62,14 @@ __device__ __forceinline__ void append_row(const LatentAppend& p, int row, float
     sq += is_q ? ss : 0.f;
     sc += is_q ? 0.f : ss;
   }
-  la_block_sum2(sq, sc, red);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    sc += __shfl_xor_sync(0xffffffffu, sc, o);
+  }
   const float inv_q = p.cq ? 1.0f / sqrtf(sq / p.q_width + p.eps) : 0.f, inv_c = 1.0f / sqrtf(sc / p.c_width + p.eps);
-  for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+#pragma unroll 4
+  for (int i = lane; i < pieces; i += 32) {
     const bool is_q = i < q_pieces;
     const int e0 = (is_q ? i : i - q_pieces) * 8;
     float v[8], w[8];
@@ -89,7 +81,7 @@ __device__ __forceinline__ void append_row(const LatentAppend& p, int row, float
     if (is_q) Vec8<TI>::store(static_cast<TI*>(p.cq) + static_cast<int64_t>(row) * p.q_rank + e0, v);
     else Vec8<TC>::store(static_cast<TC*>(p.cache) + out + e0, v);
   }
-  for (int i = threadIdx.x; i < p.s.rot / 2; i += blockDim.x) {
+  for (int i = lane; i < p.s.rot / 2; i += 32) {
     float u = la_load<TI>(p.in, r0 + 2 * i), v = la_load<TI>(p.in, r0 + 2 * i + 1);
     if (2 * i < p.s.rot_dims) {
       float sn, cs;
@@ -103,12 +95,13 @@ __device__ __forceinline__ void append_row(const LatentAppend& p, int row, float
   }
 }
 
+constexpr int AP_WARPS = 4;
 template <typename T>
-__global__ void __launch_bounds__(128) latent_append_kernel(const LatentAppend p) {
-  __shared__ float2 red[4];
+__global__ void __launch_bounds__(AP_WARPS * 32) latent_append_kernel(const LatentAppend p) {
   dependent_wait();
   dependent_trigger();
-  append_row<T, T>(p, blockIdx.x, red);
+  const int row = blockIdx.x * AP_WARPS + (threadIdx.x >> 5);
+  if (row < p.batch * p.len) append_row<T, T>(p, row);
 }
 
 static int check_shape(const LatentShape& s) {
@@ -125,7 +118,7 @@ int latent_append(const LatentAppend& a, cudaStream_t st) {
   YTC_REQUIRE(a.pos || a.pos0 + a.len <= a.cap, "latent_append: the cache is full");
   const int64_t rows = static_cast<int64_t>(a.batch) * a.len;
   YTC_CUDA(launch_overlapped(a.dtype == YTC_BF16 ? latent_append_kernel<uint16_t> : latent_append_kernel<float>,
-                             dim3(static_cast<unsigned>(rows)), dim3(128), 0, st, a));
+                             dim3(static_cast<unsigned>((rows + AP_WARPS - 1) / AP_WARPS)), dim3(AP_WARPS * 32), 0, st, a));
   count_launch();
   YTC_CUDA(cudaGetLastError());
   return YTC_OK;
@@ -178,13 +171,12 @@ __global__ void __launch_bounds__(LA_THREADS) latent_absorb_kernel(const LatentD
                                                                    int slices) {
   __shared__ float part[LA_WARPS][128];
   __shared__ float q_s[512];
-  __shared__ float2 red[LA_WARPS];
   const LatentShape& s = p.s;
   const int row = blockIdx.y;
   if (static_cast<int>(blockIdx.x) == s.heads * slices) {
     dependent_wait();
     dependent_trigger();
-    append_row<TQ, TC>(ap, row, red);
+    if (threadIdx.x < 32) append_row<TQ, TC>(ap, row);
     return;
   }
   const int h = blockIdx.x / slices, c0 = (blockIdx.x - h * slices) * cols;
