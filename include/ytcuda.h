@@ -385,7 +385,7 @@ int ytcuda_window_attn_fwd(int dtype, const void* q, const void* k, const void* 
 
 /* Router of a mixture of experts with `identity` pass-through experts behind the `experts` real ones: s = softmax(logits)
  * over both kinds (score 0) or sigmoid of every logit (score 1) is the weight of a route (used as it is), s + correction
- * (NULL: s) its selection score. The routes are split into
+ * (NULL: the logit, which has the same order) its selection score. The routes are split into
  * `groups` contiguous blocks of one size, ranked by their maximal selection score; the `top` routes with the largest
  * selection scores are taken from the `keep` leading blocks.
  * choice / weight [rows, top] in the order of choice (-1: none left); rank [rows, top]: running number of the token

@@ -34,9 +34,9 @@ def expert_ff(w, p, h, limit):
 
 
 def route(logits, top):
-    """One token's router logits [E] -> (chosen experts, their scores)."""
+    """One token's router logits [E] -> (chosen experts, their scores). (Scores have the order of the logits.)"""
     s = sigmoid(logits)
-    chosen = sorted(range(len(s)), key=lambda i: (-s[i], i))[:top]
+    chosen = sorted(range(len(s)), key=lambda i: (-logits[i], i))[:top]
     return chosen, [s[i] for i in chosen]
 
 

@@ -275,7 +275,7 @@ def linear_case(L, code, act, x, w, want, cols, limit, dtype):
 def test_sigmoid_router(L, experts, top):
     rng = np.random.default_rng(experts)
     rows = 41
-    z = (rng.standard_normal((rows, experts)) * 2).astype(np.float32)
+    z = (rng.standard_normal((rows, experts)) * np.linspace(1, 30, rows)[:, None]).astype(np.float32)  # also scores that round to 1
     zd, ch = dev(z), torch.empty(rows, top, dtype=torch.int32, device="cuda")
     rk, w, cnt = torch.empty_like(ch), torch.empty(rows, top, device="cuda"), torch.zeros(experts, dtype=torch.int32, device="cuda")
     check(L.ytcuda_moe_route(zd.data_ptr(), experts, None, rows, experts, 0, top, 1, 1, 1, ch.data_ptr(), w.data_ptr(),

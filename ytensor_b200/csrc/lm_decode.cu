@@ -685,11 +685,13 @@ __device__ __forceinline__ bool comes_before(float a, int i, float b, int j) { r
 __device__ __forceinline__ void block_route(float* s, float* c, float* g, float* red, const float* correction,
                                             const RouterSpec& r, int* choice, float* weight) {
   const int n = r.experts + r.identity;
+  if (!correction)
+    for (int i = threadIdx.x; i < n; i += DL_THREADS) c[i] = s[i];
   if (r.score == ROUTE_SIGMOID) {
     for (int i = threadIdx.x; i < n; i += DL_THREADS) {
       const float p = lm_sigmoid(s[i]);
       s[i] = p;
-      c[i] = p + correction[i];
+      if (correction) c[i] = p + correction[i];
     }
   } else {
     float m = -INFINITY;
@@ -705,7 +707,7 @@ __device__ __forceinline__ void block_route(float* s, float* c, float* g, float*
     for (int i = threadIdx.x; i < n; i += DL_THREADS) {
       const float p = s[i] / sum;
       s[i] = p;
-      c[i] = p + correction[i];
+      if (correction) c[i] = p + correction[i];
     }
   }
   if (threadIdx.x < r.top) {  // (places that no route takes)
@@ -778,7 +780,7 @@ __global__ void __launch_bounds__(DL_THREADS, 2) decode_route_kernel(const Decod
   for (int i = threadIdx.x; i < (end - begin) * 2; i += DL_THREADS)
     if (begin * 2 + i < n) st_cluster(s + begin * 2 + i, 0, sum_sub(part, i, ks));
   cluster_barrier();
-  if (rank == 0) block_route(s, c, g, red, corr, p.r, p.choice, p.weight);
+  if (rank == 0) block_route(s, c, g, red, p.correction ? corr : nullptr, p.r, p.choice, p.weight);
 }
 
 int decode_route(const DecodeRoute& a, cudaStream_t st) {

@@ -261,7 +261,8 @@ int decayed_attention(const DecayedAttn& a, cudaStream_t st);
 
 // ---------------------------------------------------------------- mixture of experts
 // `experts` experts and `identity` pass-through experts share one router: s = softmax(logits), or sigmoid of every logit,
-// decides the weights, s + correction (null: s) the selection. The routes are split into `count` contiguous blocks of one
+// decides the weights, s + correction the selection (without a correction the logits, which have the order of the scores
+// also where these round to the same number). The routes are split into `count` contiguous blocks of one
 // size, ranked by their maximal selection score; the `top` routes are taken from the `keep` leading blocks.
 enum { ROUTE_SOFTMAX = 0, ROUTE_SIGMOID = 1 };
 struct RouterSpec {
@@ -328,12 +329,12 @@ __device__ __forceinline__ void warp_route(float* s, float* c, const float* corr
                                            int& choice, float& weight) {
   const int n = r.experts + r.identity;
   const uint32_t floor = ordered_key(-INFINITY);
-  float v[VPL];
+  float v[VPL], z[VPL];
   float m = -INFINITY;
 #pragma unroll
   for (int j = 0; j < VPL; ++j) {
     const int i = j * 32 + lane;
-    v[j] = i < n ? s[i] : -INFINITY;
+    v[j] = z[j] = i < n ? s[i] : -INFINITY;
     m = fmaxf(m, v[j]);
   }
 #pragma unroll
@@ -358,7 +359,7 @@ __device__ __forceinline__ void warp_route(float* s, float* c, const float* corr
     const int i = j * 32 + lane;
     key[j] = 0;
     if (i < n) {
-      const float p = v[j] / sum, choice_score = correction ? p + correction[i] : p;
+      const float p = v[j] / sum, choice_score = correction ? p + correction[i] : z[j];
       s[i] = p;
       c[i] = choice_score;
       key[j] = ordered_key(choice_score);
