@@ -58,11 +58,12 @@ struct TcSmem {
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;
   static constexpr int B_BYTES = BN * TC_BK * 2;
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int OUT_OFFSET = TC_STAGES * STAGE_BYTES;  // staged stores: 4 warps x 32 rows x 128 bytes
-  static constexpr int BAR_OFFSET = OUT_OFFSET + 4 * TC_OUT_BYTES;
+  static constexpr int BAR_OFFSET = TC_STAGES * STAGE_BYTES;
   // full[STAGES], empty[STAGES], tmem_full[2], tmem_empty[2], tmem base word, abort word
   static constexpr int TOTAL = BAR_OFFSET + (2 * TC_STAGES + 4) * 8 + 16;
   static constexpr int DYN_BYTES = TOTAL + 1024;  // slack to align the ring to 1024 B
+  static constexpr int OUT_OFFSET = (TOTAL + 127) / 128 * 128;  // staged stores: the epilogue warps' areas
+  static constexpr int DYN_STAGED = OUT_OFFSET + 4 * TC_OUT_BYTES + 1024;
 };
 
 template <int BN, int OUT_DT>
@@ -511,10 +512,11 @@ struct Tc2Smem {
   static constexpr int A_BYTES = TC_BM * TC_BK * 2;         // 128 rows of A
   static constexpr int B_BYTES = (TC2_BN / 2) * TC_BK * 2;  // 128 columns of B
   static constexpr int STAGE_BYTES = A_BYTES + B_BYTES;
-  static constexpr int OUT_OFFSET = TC2_STAGES * STAGE_BYTES;
-  static constexpr int BAR_OFFSET = OUT_OFFSET + 4 * TC_OUT_BYTES;
+  static constexpr int BAR_OFFSET = TC2_STAGES * STAGE_BYTES;
   static constexpr int TOTAL = BAR_OFFSET + (2 * TC2_STAGES + 4) * 8 + 16;
   static constexpr int DYN_BYTES = TOTAL + 1024;
+  static constexpr int OUT_OFFSET = (TOTAL + 127) / 128 * 128;
+  static constexpr int DYN_STAGED = OUT_OFFSET + 4 * TC_OUT_BYTES + 1024;
 };
 
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(TC_THREADS, 1)
@@ -1001,13 +1003,14 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
     p.tiles_m = (m + 255) / 256;
     p.tiles_n = (n + TC2_BN - 1) / TC2_BN;
     p.total_tiles = static_cast<int>(static_cast<int64_t>(p.tiles_m) * p.tiles_n * batch);
+    const int smem = p.staged ? Tc2Smem::DYN_STAGED : Tc2Smem::DYN_BYTES;
     int clusters = sm_count() / 2;
     if (clusters > p.total_tiles) clusters = p.total_tiles;
     {
-      const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc2_kernel), Tc2Smem::DYN_BYTES);
+      const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc2_kernel), smem);
       if (s != YTC_OK) return s;
     }
-    YTC_CUDA(launch_overlapped(gemm_tc2_kernel, dim3(clusters * 2), dim3(TC_THREADS), Tc2Smem::DYN_BYTES, st, tmA, tmB, p));
+    YTC_CUDA(launch_overlapped(gemm_tc2_kernel, dim3(clusters * 2), dim3(TC_THREADS), smem, st, tmA, tmB, p));
     count_launch();
     YTC_CUDA(cudaGetLastError());
     return YTC_OK;
@@ -1020,13 +1023,15 @@ static int launch_tc(int dtype_in, int dtype_out, const void* A, const void* B, 
     p.tile_live = live;
   }
   if (BN == 256) {
-    const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc_kernel<256>), TcSmem<256>::DYN_BYTES);
+    const int smem = p.staged ? TcSmem<256>::DYN_STAGED : TcSmem<256>::DYN_BYTES;
+    const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc_kernel<256>), smem);
     if (s != YTC_OK) return s;
-    YTC_CUDA(launch_overlapped(gemm_tc_kernel<256>, dim3(grid), dim3(TC_THREADS), TcSmem<256>::DYN_BYTES, st, tmA, tmB, p));
+    YTC_CUDA(launch_overlapped(gemm_tc_kernel<256>, dim3(grid), dim3(TC_THREADS), smem, st, tmA, tmB, p));
   } else {
-    const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc_kernel<128>), TcSmem<128>::DYN_BYTES);
+    const int smem = p.staged ? TcSmem<128>::DYN_STAGED : TcSmem<128>::DYN_BYTES;
+    const int s = ensure_dynamic_smem(reinterpret_cast<const void*>(gemm_tc_kernel<128>), smem);
     if (s != YTC_OK) return s;
-    YTC_CUDA(launch_overlapped(gemm_tc_kernel<128>, dim3(grid), dim3(TC_THREADS), TcSmem<128>::DYN_BYTES, st, tmA, tmB, p));
+    YTC_CUDA(launch_overlapped(gemm_tc_kernel<128>, dim3(grid), dim3(TC_THREADS), smem, st, tmA, tmB, p));
   }
   count_launch();
   if (live) cudaFreeAsync(live, st);
